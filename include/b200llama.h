@@ -23,7 +23,10 @@ extern "C" {
 enum { B200_TYPE_F32 = 0, B200_TYPE_Q8_0 = 8, B200_TYPE_Q4_K = 12, B200_TYPE_Q6_K = 14 };
 /* KV cache element types: FP32 (KVCacheLayer::k_dev_fp32, model.h:137-138) or INT8 with one FP32
  * scale per (position, kv head) (k_dev_quantized / k_dev_scales, model.h:140-143). */
-enum { B200_KV_F32 = 0, B200_KV_I8 = 1 };
+enum { B200_KV_F32 = 0, B200_KV_I8 = 1, B200_KV_BF16 = 2 /* block models in bfloat16; reported, not chosen */ };
+/* What a model folder's engine computes in: bfloat16 matrix products and cache with FP32 accumulation (norms, attention
+ * scores and weights, the residual stream, recurrences and their gates stay FP32), or FP32 throughout. */
+enum { B200_DTYPE_BF16 = 0, B200_DTYPE_F32 = 1 };
 
 typedef struct b200_engine b200_engine;
 
@@ -65,6 +68,12 @@ int b200_engine_finalize(b200_engine* e);
 /* Parses a GGUF file (gguf_parser.cpp:123) and does create + upload + finalize. desc_overrides may be
  * NULL; when given, only kv_dtype, max_seqs, max_ctx, act_planes, device and the tp_* fields are read. */
 int b200_engine_load_gguf(const char* path, const b200_model_desc* desc_overrides, b200_engine** out);
+/* The same for any model the registry knows: a GGUF file (as above; dtype is not used), or a folder with config.json and
+ * model.safetensors (bfloat16 weights) whose "architecture" names a block model. desc_overrides may be NULL; of it, max_seqs, max_ctx
+ * (0 = 4096) and device are read. Such an engine serves every entry point below that takes an engine, with these
+ * differences: a slot continues where it stands (a call's start position is the number of tokens the slot holds, or 0 to
+ * start over; anything else is refused), tensors are not uploaded one by one, and tensor parallelism is not built. */
+int b200_engine_load_model(const char* path, int dtype, const b200_model_desc* desc_overrides, b200_engine** out);
 int b200_engine_get_desc(const b200_engine* e, b200_model_desc* out);
 int b200_engine_destroy(b200_engine* e);
 
@@ -96,6 +105,10 @@ int b200_prefill(b200_engine* e, int seq_slot, const int32_t* token_ids, int n, 
  * per-token arithmetic as one b200_prefill call per sequence on the tensor-core path (n >= 16). */
 int b200_prefill_batch(b200_engine* e, int n_seqs, const int32_t* slots, const int32_t* token_ids, const int32_t* lens,
                        const int32_t* start_pos, float* host_logits_last);
+/* Prompt ingestion with the logits of chosen tokens: want[i] (0 .. n-1) names a token of this call, host_logits [n_want][vocab]
+ * receives their logits in that order. Always the tensor-core path, for any n >= 1. */
+int b200_prefill_rows(b200_engine* e, int seq_slot, const int32_t* token_ids, int n, int start_pos, const int32_t* want, int n_want,
+                      float* host_logits);
 /* The chunk plan b200_prefill_batch follows for prompts of these lengths (host arithmetic only, no GPU needed): one
  * record per run of tokens, out[i] = {chunk, first row in the chunk, tokens, position of the first token, index of the
  * sequence whose prompt ends with this run or -1}. chunk = tokens per chunk (the engine uses 512). */

@@ -11,6 +11,7 @@ CSRC = os.path.join(os.path.dirname(os.path.abspath(__file__)), "csrc")
 LIB_ENGINE = os.path.join(CSRC, "libb200llama.so")
 LIB_SYNTH = os.path.join(CSRC, "libb200synth.so")
 
+ENGINE_SOURCES = ["engine.cu", "gguf.cpp", "safetensors.cpp", "model_registry.cpp"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "-Xcompiler", "-fPIC", "-shared"]
 
@@ -36,8 +37,9 @@ def build_engine(force=False, verbose=False):
         return LIB_ENGINE
     nvcc = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
     cmd = [nvcc] + NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else []) + \
-          ["-o", LIB_ENGINE, os.path.join(CSRC, "engine.cu"), os.path.join(CSRC, "gguf.cpp"), "-ldl"]
+          ["-o", LIB_ENGINE + f".{os.getpid()}"] + [os.path.join(CSRC, f) for f in ENGINE_SOURCES] + ["-ldl"]
     subprocess.run(cmd, check=True, cwd=CSRC)
+    os.replace(LIB_ENGINE + f".{os.getpid()}", LIB_ENGINE)  # whole or not at all
     return LIB_ENGINE
 
 

@@ -7,7 +7,8 @@ import numpy as np
 
 from . import _build
 
-KV_F32, KV_I8 = 0, 1
+KV_F32, KV_I8, KV_BF16 = 0, 1, 2
+DTYPES = {"bfloat16": 0, "float32": 1}
 
 
 class B200Error(RuntimeError):
@@ -27,8 +28,8 @@ class ModelDesc(ctypes.Structure):
 
 EXPORTS = [
     "b200_last_error", "b200_device_count", "b200_engine_create", "b200_engine_upload_tensor",
-    "b200_engine_finalize", "b200_engine_load_gguf", "b200_engine_get_desc", "b200_engine_destroy",
-    "b200_kv_reset", "b200_lookup_embedding", "b200_forward", "b200_prefill", "b200_prefill_batch", "b200_prefill_plan", "b200_decode",
+    "b200_engine_finalize", "b200_engine_load_gguf", "b200_engine_load_model", "b200_engine_get_desc", "b200_engine_destroy",
+    "b200_kv_reset", "b200_lookup_embedding", "b200_forward", "b200_prefill", "b200_prefill_rows", "b200_prefill_batch", "b200_prefill_plan", "b200_decode",
     "b200_generate_greedy", "b200_generate_greedy_penalized", "b200_dequant", "b200_matvec", "b200_matmul", "b200_rmsnorm", "b200_rmsnorm_batch",
     "b200_fused_qkv_rope", "b200_fused_gate_up_swiglu", "b200_attention_decode", "b200_attention_prefill",
     "b200_attention_decode_noalloc", "b200_engine_stats", "b200_engine_time_kernel", "b200_engine_read_trace",
@@ -53,12 +54,14 @@ def lib():
     L.b200_engine_upload_tensor.argtypes = [_vp, ctypes.c_char_p, _i, _vp, _sz, _i64, _i64]
     L.b200_engine_finalize.argtypes = [_vp]
     L.b200_engine_load_gguf.argtypes = [ctypes.c_char_p, ctypes.POINTER(ModelDesc), ctypes.POINTER(_vp)]
+    L.b200_engine_load_model.argtypes = [ctypes.c_char_p, _i, ctypes.POINTER(ModelDesc), ctypes.POINTER(_vp)]
     L.b200_engine_get_desc.argtypes = [_vp, ctypes.POINTER(ModelDesc)]
     L.b200_engine_destroy.argtypes = [_vp]
     L.b200_kv_reset.argtypes = [_vp, _i]
     L.b200_lookup_embedding.argtypes = [_vp, _i, _vp]
     L.b200_forward.argtypes = [_vp, _i, _vp, _i, _vp]
     L.b200_prefill.argtypes = [_vp, _i, _vp, _i, _i, _vp]
+    L.b200_prefill_rows.argtypes = [_vp, _i, _vp, _i, _i, _vp, _i, _vp]
     L.b200_decode.argtypes = [_vp, _i, _vp, _vp, _vp, _vp, _vp]
     L.b200_prefill_batch.argtypes = [_vp, _i, _vp, _vp, _vp, _vp, _vp]
     L.b200_prefill_plan.argtypes = [_i, _vp, _i, _vp, _i, ctypes.POINTER(_i)]
@@ -128,6 +131,14 @@ class Engine:
         return cls(h.value)
 
     @classmethod
+    def from_model(cls, path, dtype="bfloat16", max_seqs=1, max_ctx=0, device=0):
+        """Any model the registry knows: a GGUF file, or a folder with config.json and model.safetensors."""
+        ov = ModelDesc(max_seqs=max_seqs, max_ctx=max_ctx, device=device, tp_size=1)
+        h = _vp()
+        _check(lib().b200_engine_load_model(os.fsencode(path), DTYPES[dtype], ctypes.byref(ov), ctypes.byref(h)))
+        return cls(h.value)
+
+    @classmethod
     def create(cls, cfg, kv_dtype=KV_F32, max_seqs=1, max_ctx=0, act_planes=3, device=0):
         d = ModelDesc(cfg["hidden"], cfg["ffn"], cfg["n_heads"], cfg["n_kv_heads"], cfg["n_layers"], cfg["vocab"],
                       cfg["max_pos"], cfg.get("eps", 1e-5), cfg["theta"], kv_dtype, max_seqs, max_ctx, act_planes,
@@ -174,6 +185,13 @@ class Engine:
         ids = _i32(ids)
         logits = np.empty(self.vocab, np.float32) if want_logits else None
         _check(lib().b200_prefill(self._h, slot, _ptr(ids), len(ids), start_pos, _ptr(logits)))
+        return logits
+
+    def prefill_rows(self, ids, want, slot=0, start_pos=0):
+        """Ingests ids and returns the logits [len(want)][vocab] of the tokens at places `want` among them."""
+        ids, want = _i32(ids), _i32(want)
+        logits = np.empty((len(want), self.vocab), np.float32)
+        _check(lib().b200_prefill_rows(self._h, slot, _ptr(ids), len(ids), start_pos, _ptr(want), len(want), _ptr(logits)))
         return logits
 
     def prefill_batch(self, prompts, slots=None, start_pos=None, want_logits=True):

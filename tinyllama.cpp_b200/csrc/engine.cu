@@ -1,6 +1,8 @@
 // Engine: weight residency, KV cache, the per-token launch sequence and its CUDA graph.
 #include "engine.h"
 
+#include <sys/stat.h>
+
 #include <algorithm>
 #include <cmath>
 #include <cstdio>
@@ -10,12 +12,16 @@
 #include "attn.cuh"
 #include "attn_cluster.cuh"
 #include "attn_prefill.cuh"
+#include "block_model.h"
+#include "dense_gemm.cuh"
 #include "dequant.cuh"
 #include "gemv.cuh"
 #include "gemm_tc.cuh"
 #include "gguf.h"
+#include "latent_attn.cuh"
 #include "misc.cuh"
 #include "tp.h"
+#include "wkv.cuh"
 
 namespace b200 {
 
@@ -471,6 +477,20 @@ static int tp_reduce_add(b200_engine* e, int batch, cudaStream_t st, float* h = 
   return 2;
 }
 
+// A run of consecutive tokens of one sequence inside a chunk: rows [row0, row0 + len) of the chunk's buffers hold the
+// tokens at positions start .. start+len-1 of KV slot `slot`. logits_to >= 0: this run ends the prompt
+// of sequence logits_to.
+struct PrefillRun {
+  int row0, len, slot, start, logits_to;
+};
+
+// A row of the chunk whose logits are wanted, and the row of the caller's host buffer they go to.
+struct WantedRow {
+  int row, out;
+};
+
+#include "block_engine.inc"
+
 // One fused linear layer of the step: the matvec kernel (one launch column per sequence), or, for
 // large batches on a single GPU, fp16 conversion (+RMSNorm) followed by the tensor-core matmul.
 // Returns the number of launches; *grid_out = partial-argmax parts per sequence (lm_head only).
@@ -518,11 +538,14 @@ static int launch_linear(b200_engine* e, GemvParams p, int batch, cudaStream_t s
   return n;
 }
 
-// The launch sequence of one decode step for `batch` sequences (also what gets captured).
-// Per layer: [RMSNorm + QKV + RoPE] -> [KV append + attention] -> [O proj + residual] ->
+// Argmax packets of the lm_head launch, behind the exchange slots: [rank][batch][parts].
+static uint2* amax_packets(const b200_engine* e, void* region) { return static_cast<uint2*>(region) + (size_t)2 * e->tp_size * e->max_seqs * e->H; }
+
+// The launches of a packed-weight (GGUF) model's decode step up to the logits and their argmax partials; *head_parts =
+// partials per sequence. Per layer: [RMSNorm + QKV + RoPE] -> [KV append + attention] -> [O proj + residual] ->
 // [RMSNorm + gate/up + SwiGLU] -> [down proj + residual]; then [RMSNorm + lm_head + argmax
-// partials] and token selection. Returns the number of kernel launches.
-static int enqueue_step(b200_engine* e, int batch, int nsplit, cudaStream_t st, bool with_embed, int* head_ctas_out, bool penalized = false) {
+// partials]. Returns the number of kernel launches.
+static int packed_forward_step(b200_engine* e, int batch, int nsplit, cudaStream_t st, bool with_embed, bool penalized, int* head_parts) {
   int launches = 0;
   const int H = e->H, F = e->F, KVD = e->KVD;
   const float eps = std::max(e->desc.rms_norm_eps, 1e-5f);  // reference utils.cpp:666-667
@@ -536,9 +559,6 @@ static int enqueue_step(b200_engine* e, int batch, int nsplit, cudaStream_t st, 
   const bool peer = tp && e->use_peer && !use_tc;
   auto slot_of = [&](void* region, int k, int src) {
     return static_cast<uint2*>(region) + ((size_t)(k & 1) * e->tp_size + src) * e->max_seqs * H;
-  };
-  auto amax_of = [&](void* region) {  // argmax packets of the lm_head launch, behind the exchange slots: [rank][batch][parts]
-    return static_cast<uint2*>(region) + (size_t)2 * e->tp_size * e->max_seqs * H;
   };
   float* hcur = e->d_h;
   float* hnext = e->d_h2;
@@ -654,7 +674,7 @@ static int enqueue_step(b200_engine* e, int batch, int nsplit, cudaStream_t st, 
     const int head_grid = std::max(1, std::min(e->out_w.tiles, e->num_sms));
     const unsigned head_epoch_k = 2u * (unsigned)e->L + 1u;
     if (peer) {
-      for (int r = 0; r < e->tp_size; ++r) p.amax_peer[r] = amax_of(e->peer_region[r]) + (size_t)e->tp_rank * batch * head_grid;
+      for (int r = 0; r < e->tp_size; ++r) p.amax_peer[r] = amax_packets(e, e->peer_region[r]) + (size_t)e->tp_rank * batch * head_grid;
       p.tp = e->tp_size; p.tp_rank = e->tp_rank;
       p.epoch_base = e->d_epoch;
       p.amax_epoch_k = head_epoch_k;
@@ -669,21 +689,36 @@ static int enqueue_step(b200_engine* e, int batch, int nsplit, cudaStream_t st, 
       n.check(n.AllGather(p.amax_idx, e->d_amax_idx, (size_t)batch * grid, Nccl::kInt32, e->nccl_comm, st), "ncclAllGather");
       launches += 3;
     }
-    if (head_ctas_out) *head_ctas_out = grid;
-    SelectParams s{};
-    s.amax_val = e->d_amax_val; s.amax_idx = e->d_amax_idx; s.nparts = grid * e->tp_size; s.parts_per_rank = grid; s.batch = batch;
-    s.tokens = e->d_tokens; s.positions = e->d_positions; s.argmax_out = e->d_argmax; s.step_counter = e->d_step;
-    s.forced = e->d_forced; s.forced_steps = e->d_forced_steps; s.log = e->d_log; s.log_cap = e->log_cap;
-    if (penalized) { s.pen_ring = e->d_pen_ring; s.pen_count = e->d_pen_count; s.pen_counts = e->d_pen_counts; s.pen_stride = e->pen_stride; }
-    if (peer) {  // the next step's packets carry new numbers
-      s.epoch = e->d_epoch; s.epoch_inc = 2u * (unsigned)e->L + 2u;
-      s.amax_pkts = amax_of(e->xregion); s.epoch_k = head_epoch_k; s.error_flag = e->d_error;
-    }
-    select_kernel<<<1, 256, 0, st>>>(s);
-    CK(cudaGetLastError());
-    ++launches;
+    *head_parts = grid;
   }
   return launches;
+}
+
+// The launch sequence of one decode step for `batch` sequences (also what gets captured): the model's layers and
+// logits, then token selection. Returns the number of kernel launches.
+static int enqueue_step(b200_engine* e, int batch, int nsplit, cudaStream_t st, bool with_embed, int* head_ctas_out, bool penalized = false) {
+  const bool rows = batch >= e->gemm_min_batch;
+  const bool peer = e->tp_size > 1 && e->use_peer && !rows;
+  int parts = 0, launches;
+  if (e->blocks) {
+    if (rows && penalized) throw std::runtime_error("the repetition penalty of the device loop is built for the matvec path (batch < " + std::to_string(e->gemm_min_batch) + ")");
+    launches = rows ? block_forward_batch(e, batch, st, with_embed, &parts) : block_forward_step(e, batch, st, with_embed, penalized, &parts);
+  } else {
+    launches = packed_forward_step(e, batch, nsplit, st, with_embed, penalized, &parts);
+  }
+  if (head_ctas_out) *head_ctas_out = parts;
+  SelectParams s{};
+  s.amax_val = e->d_amax_val; s.amax_idx = e->d_amax_idx; s.nparts = parts * e->tp_size; s.parts_per_rank = parts; s.batch = batch;
+  s.tokens = e->d_tokens; s.positions = e->d_positions; s.argmax_out = e->d_argmax; s.step_counter = e->d_step;
+  s.forced = e->d_forced; s.forced_steps = e->d_forced_steps; s.log = e->d_log; s.log_cap = e->log_cap;
+  if (penalized) { s.pen_ring = e->d_pen_ring; s.pen_count = e->d_pen_count; s.pen_counts = e->d_pen_counts; s.pen_stride = e->pen_stride; }
+  if (peer) {  // the next step's packets carry new numbers
+    s.epoch = e->d_epoch; s.epoch_inc = 2u * (unsigned)e->L + 2u;
+    s.amax_pkts = amax_packets(e, e->xregion); s.epoch_k = 2u * (unsigned)e->L + 1u; s.error_flag = e->d_error;
+  }
+  select_kernel<<<1, 256, 0, st>>>(s);
+  CK(cudaGetLastError());
+  return launches + 1;
 }
 
 // ---- prompt ingestion on the tensor cores -------------------------------------------------------
@@ -716,19 +751,14 @@ static void ensure_prefill_buffers(b200_engine* e) {
   e->pf_cap = T;
 }
 
-// A run of consecutive tokens of one sequence inside a chunk: rows [row0, row0 + len) of the chunk's buffers hold the
-// tokens at positions start .. start+len-1 of KV slot `slot`. logits_to >= 0: this run ends its sequence's prompt,
-// and the logits of its last token go to row logits_to of the caller's host buffer.
-struct PrefillRun {
-  int row0, len, slot, start, logits_to;
-};
-
 // One chunk of T <= PF_CHUNK prompt tokens, possibly of several sequences (sequence-aware: every token carries its
 // own position and KV slot through the RoPE epilogue and the cache append, and attention runs per run of tokens,
 // each over its own sequence's cache rows; reference api.cpp:1144-1421 / cpu_attention.cpp:203-325).
-// meta = token ids | positions | slots, T each. After the layers, the logits of the last token of every run with
-// logits_to >= 0 are computed and copied to host_logits + logits_to * V (nullptr: left in e->d_logits only).
-static void prefill_chunk(b200_engine* e, int T, const std::vector<int>& meta, const std::vector<PrefillRun>& runs, float* host_logits) {
+// meta = token ids | positions | slots, T each. After the layers, the logits of the wanted rows are computed and copied
+// to row `out` of host_logits (nullptr: those of the last one are left in e->d_logits).
+static void prefill_chunk(b200_engine* e, int T, const std::vector<int>& meta, const std::vector<PrefillRun>& runs, const std::vector<WantedRow>& wanted,
+                          float* host_logits) {
+  if (e->blocks) return block_prefill_chunk(e, T, meta, runs, wanted, host_logits);
   ensure_prefill_buffers(e);
   cudaStream_t st = e->stream;
   const int H = e->H, F = e->F, KVD = e->KVD;
@@ -798,23 +828,23 @@ static void prefill_chunk(b200_engine* e, int T, const std::vector<int>& meta, c
       if (tp) tp_reduce_add(e, T, st, e->pf_h, e->pf_partial);
     }
   }
-  for (const PrefillRun& r : runs) {  // final norm + lm_head for the last token of a prompt only, on the matvec kernel
-    if (r.logits_to < 0) continue;
+  for (const WantedRow& r : wanted) {  // final norm + lm_head for the wanted rows only, on the matvec kernel
     GemvParams p{};
-    p.seg[0] = seg_of(e->out_w); p.nseg = 1; p.K = H; p.x = e->pf_h + (size_t)(r.row0 + r.len - 1) * H; p.x_stride = H;
+    p.seg[0] = seg_of(e->out_w); p.nseg = 1; p.K = H; p.x = e->pf_h + (size_t)r.row * H; p.x_stride = H;
     p.norm_w = e->out_norm.f32(); p.eps = eps; p.epi = EPI_STORE; p.y = tp ? e->d_logits_local : e->d_logits; p.y_stride = e->Vl;
     launch_gemv(e, p, 1, st);
     if (tp) {  // every rank holds its share of the vocabulary: gather the shares (in rank order = vocabulary order for one row)
       Nccl& n = Nccl::get();
       n.check(n.AllGather(e->d_logits_local, e->d_logits, (size_t)e->Vl, Nccl::kFloat32, e->nccl_comm, st), "ncclAllGather");
     }
-    if (host_logits) CK(cudaMemcpyAsync(host_logits + (size_t)r.logits_to * e->V, e->d_logits, (size_t)e->V * 4, cudaMemcpyDeviceToHost, st));
+    if (host_logits) CK(cudaMemcpyAsync(host_logits + (size_t)r.out * e->V, e->d_logits, (size_t)e->V * 4, cudaMemcpyDeviceToHost, st));
   }
 }
 
 // Prompt ingestion of one or several sequences through the tensor-core path: the tokens of all sequences are laid
-// end to end and cut into chunks of PF_CHUNK, so that short prompts share a chunk (and its weight traffic).
-// host_logits: [n_seqs][V] or nullptr.
+// end to end and cut into chunks, so that short prompts share a chunk (and its weight traffic).
+// Without `want`, host_logits [n_seqs][V] (or nullptr) receives the logits after each prompt. With it (one sequence),
+// host_logits [n_want][V] receives those of tokens want[i] of the call.
 // The chunk plan of a sequence-aware ingestion: the prompts laid end to end and cut every `chunk` tokens. Each run is
 // a stretch of one sequence inside one chunk; runs are returned in order, `chunk_of[i]` = the chunk run i belongs to.
 // Pure host arithmetic (exposed through b200_prefill_plan so that it can be checked without a GPU).
@@ -835,10 +865,10 @@ static void plan_prefill_runs(int n_seqs, const int32_t* slots, const int32_t* l
 }
 
 static void prefill_sequences(b200_engine* e, int n_seqs, const int32_t* slots, const int32_t* ids, const int32_t* lens, const int32_t* start_pos,
-                              float* host_logits) {
+                              float* host_logits, const int32_t* want = nullptr, int n_want = 0) {
   std::vector<PrefillRun> all;
   std::vector<int> chunk_of;
-  plan_prefill_runs(n_seqs, slots, lens, start_pos, PF_CHUNK, all, chunk_of);
+  plan_prefill_runs(n_seqs, slots, lens, start_pos, e->blocks ? e->blocks->chunk : PF_CHUNK, all, chunk_of);
   std::vector<size_t> seq_off(n_seqs + 1, 0);
   for (int s = 0; s < n_seqs; ++s) seq_off[s + 1] = seq_off[s] + (size_t)lens[s];
   // which sequence a run belongs to: runs come in sequence order, a new sequence starts when the previous one's last run ended
@@ -847,6 +877,7 @@ static void prefill_sequences(b200_engine* e, int n_seqs, const int32_t* slots, 
   while (i < all.size()) {
     const int c = chunk_of[i];
     std::vector<PrefillRun> runs;
+    std::vector<WantedRow> wanted;
     std::vector<int> tok, pos, slot;
     for (; i < all.size() && chunk_of[i] == c; ++i) {
       const PrefillRun& r = all[i];
@@ -856,6 +887,9 @@ static void prefill_sequences(b200_engine* e, int n_seqs, const int32_t* slots, 
         pos.push_back(r.start + t);
         slot.push_back(r.slot);
       }
+      if (!want && r.logits_to >= 0) wanted.push_back({r.row0 + r.len - 1, r.logits_to});
+      for (int i = 0; i < n_want; ++i)
+        if (want[i] >= done && want[i] < done + r.len) wanted.push_back({r.row0 + want[i] - done, i});
       done += r.len;
       if (done == lens[seq]) { ++seq; done = 0; }
     }
@@ -865,7 +899,7 @@ static void prefill_sequences(b200_engine* e, int n_seqs, const int32_t* slots, 
     meta.insert(meta.end(), tok.begin(), tok.end());
     meta.insert(meta.end(), pos.begin(), pos.end());
     meta.insert(meta.end(), slot.begin(), slot.end());
-    prefill_chunk(e, T, meta, runs, host_logits);
+    prefill_chunk(e, T, meta, runs, wanted, host_logits);
   }
 }
 
@@ -874,7 +908,7 @@ static StepGraph& get_graph(b200_engine* e, int batch, bool with_embed = true, b
   auto it = e->graphs.find(key);
   if (it != e->graphs.end()) return it->second;
   StepGraph g;
-  g.nsplit = attn_nsplit(e, batch);
+  g.nsplit = e->blocks ? 1 : attn_nsplit(e, batch);
   cudaGraph_t graph = nullptr;
   CK(cudaStreamBeginCapture(e->stream, cudaStreamCaptureModeThreadLocal));
   try {

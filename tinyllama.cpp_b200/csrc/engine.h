@@ -22,6 +22,8 @@ struct DevTensor {
   const float* f32() const { return reinterpret_cast<const float*>(base); }
 };
 
+struct BlockModel;  // block_model.h
+
 struct LayerW {
   DevTensor attn_norm, wq, wk, wv, wo, ffn_norm, wgu /* gate and up, interleaved by 8 rows */, wdown;
   void* k_cache = nullptr;
@@ -68,6 +70,7 @@ struct b200_engine {
   cudaStream_t stream = nullptr;
   std::vector<b200::LayerW> layers;
   b200::DevTensor tok_embd, out_norm, out_w;
+  b200::BlockModel* blocks = nullptr;  // set: a block model (layers above stay empty)
   float* rope = nullptr;
   // step buffers
   int* d_tokens = nullptr;

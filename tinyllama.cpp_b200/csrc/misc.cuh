@@ -90,6 +90,7 @@ __global__ void select_kernel(const SelectParams p) {
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
     }
+    if (bi == 0x7fffffff) bi = 0;  // no logit compared greater than -infinity (all NaN): a valid id all the same
     if (p.pen_ring && lane == 0) {
       // the chosen id enters the window of generated tokens, the id generated PEN_WINDOW steps ago leaves it
       int* ring = p.pen_ring + (size_t)b * PEN_WINDOW;

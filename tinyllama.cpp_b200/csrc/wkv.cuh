@@ -1,0 +1,217 @@
+// WKV mixer: the recurrence S <- diag(w_t) S + k_t v_t^T per head (S is key x value, FP32), read out before the update
+// with a bonus for the current token: o_t = (S + diag(u) k_t v_t^T)^T r_t. Everything here is FP32.
+//
+//   wkv_step_kernel  one token of several sequences (decode): one block per (head, sequence); the decay's second matrix
+//                    product, the recurrence, the head norm and the gate in one launch
+//   wkv_scan_kernel  runs of tokens (prompts): the value columns of a head are independent of one another, so a block
+//                    takes a few columns of one head, keeps their state in registers (eight keys per thread) and walks
+//                    the run's tokens, whose r, k, w, v pieces arrive in shared memory a tile ahead (cp.async)
+//
+// State of a slot: [head][key][value]. A token at position 0 starts from zeros whatever the slot held before.
+#pragma once
+#include "block_rows.cuh"
+
+namespace b200 {
+
+constexpr int WKV_STEP_THREADS = 256;
+constexpr int WKV_MAX_DIM = 256;
+
+struct WkvStepParams {
+  const float* rkvg;      // [batch][stride]: r, k, v, gate at offsets 0, hd, 2 hd, 3 hd (hd = padded heads * dim)
+  int stride, off;        // off = hd
+  const float* low;       // [batch][low_stride] inner vector of the decay product
+  int low_stride, rank;
+  const __nv_bfloat16* w2;  // [heads * dim][pad8(rank)]
+  const float* w0;
+  const float* u;
+  const float* norm;
+  float eps;
+  float* state;           // [slot][heads][dim][dim]
+  const int* slots;
+  const int* positions;
+  int heads, dim;
+  void* out;              // [batch][out_stride]
+  int out_stride;
+};
+
+template <typename A>
+__global__ void __launch_bounds__(WKV_STEP_THREADS) wkv_step_kernel(const WkvStepParams p) {
+  __shared__ float r_s[WKV_MAX_DIM], k_s[WKV_MAX_DIM], w_s[WKV_MAX_DIM], part[WKV_STEP_THREADS], red[WKV_STEP_THREADS / 32];
+  const int tid = threadIdx.x, h = blockIdx.x, b = blockIdx.y, D = p.dim, hc = h * D;
+  pdl_launch_dependents();
+  pdl_wait();
+  const float* in = p.rkvg + (size_t)b * p.stride + hc;
+  const int pos = p.positions[b];
+  float* S = p.state + ((size_t)p.slots[b] * p.heads + h) * D * D;
+  const int groups = WKV_STEP_THREADS / D;  // key groups working side by side on every value column
+  const int col = tid % D, grp = tid / D;
+  const bool active = grp < groups;
+  constexpr int KEEP = 16;  // state elements per thread held in registers (all of them up to dim 64)
+  float st[KEEP];
+  if (active && pos > 0) {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int k = grp + i * groups;
+      st[i] = k < D ? S[(size_t)k * D + col] : 0.f;
+    }
+  } else {
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) st[i] = 0.f;
+  }
+  if (tid < D) {
+    r_s[tid] = in[tid];
+    k_s[tid] = in[p.off + tid];
+    float acc = p.w0[hc + tid];
+    const __nv_bfloat16* w2 = p.w2 + (size_t)(hc + tid) * pad8(p.rank);
+    const float* low = p.low + (size_t)b * p.low_stride;
+#pragma unroll 8
+    for (int j = 0; j < p.rank; ++j) acc = fmaf(__bfloat162float(w2[j]), low[j], acc);
+    w_s[tid] = expf(-expf(acc));
+  }
+  __syncthreads();
+  float o = 0.f;
+  if (active) {
+    const float v = in[2 * p.off + col];
+    auto one = [&](int k, float s) -> float {
+      const float kv = k_s[k] * v;
+      o = fmaf(r_s[k], fmaf(p.u[hc + k], kv, s), o);
+      return fmaf(w_s[k], s, kv);
+    };
+#pragma unroll
+    for (int i = 0; i < KEEP; ++i) {
+      const int k = grp + i * groups;
+      if (k < D) S[(size_t)k * D + col] = one(k, st[i]);
+    }
+    for (int k = grp + KEEP * groups; k < D; k += groups) S[(size_t)k * D + col] = one(k, pos > 0 ? S[(size_t)k * D + col] : 0.f);
+    part[grp * D + col] = o;
+  }
+  __syncthreads();
+  float tot = 0.f;
+  if (tid < D)
+    for (int g = 0; g < groups; ++g) tot += part[g * D + tid];
+  float ss[1] = {tot * tot};
+  block_sums<1, WKV_STEP_THREADS / 32>(ss, red);
+  if (tid < D)
+    static_cast<A*>(p.out)[(size_t)b * p.out_stride + hc + tid] =
+        to_operand<A>(tot * (1.0f / sqrtf(ss[0] / (float)D + p.eps)) * p.norm[hc + tid] * in[3 * p.off + tid]);
+}
+
+constexpr int WKV_SCAN_THREADS = 128;
+constexpr int WKV_TILE = 16;  // tokens staged per step
+constexpr int WKV_KPT = 8;    // keys per thread
+
+struct WkvScanParams {
+  const float* rkv;    // [T][stride]: r, k, v at offsets 0, off, 2 off
+  int stride, off;
+  const float* decay;  // [T][decay_stride]
+  int decay_stride;
+  const float* u;      // [heads * dim]
+  float* state;        // [slot][heads][dim][dim]
+  const RunDesc* runs;
+  int heads, dim;
+  float* o;            // [T][o_stride]
+  int o_stride;
+  // the row the next run's token shift starts from: h of the run's last token
+  const float* h;
+  int h_stride, W;
+  float* shift;        // [slot][2][shift_stride]
+  int shift_stride;
+};
+
+// lanes per value column: a power of two with lanes * WKV_KPT >= dim
+__host__ __device__ __forceinline__ int wkv_lanes(int dim) {
+  int l = 1;
+  while (l * WKV_KPT < dim) l *= 2;
+  return l;
+}
+__host__ __device__ __forceinline__ int wkv_cols(int dim) { return WKV_SCAN_THREADS / wkv_lanes(dim); }
+__host__ __device__ __forceinline__ size_t wkv_scan_smem(int dim) {
+  return (size_t)2 * WKV_TILE * (3 * wkv_lanes(dim) * WKV_KPT + wkv_cols(dim)) * 4;
+}
+
+// grid = (column blocks of a head, heads, runs). L = lanes per column.
+template <int L>
+__global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvScanParams p) {
+  extern __shared__ __align__(16) float scan_s[];  // two tiles of [token][r | k | w (DP each) | v (cols)]
+  constexpr int DP = L * WKV_KPT, COLS = WKV_SCAN_THREADS / L, ROW = 3 * DP + COLS;
+  const int tid = threadIdx.x, h = blockIdx.y, D = p.dim, hc = h * D;
+  const RunDesc run = p.runs[blockIdx.z];
+  const int ln = tid % L, col = blockIdx.x * COLS + tid / L;
+  const bool col_ok = col < D;
+  const int k0 = ln * WKV_KPT;
+  float* S = p.state + ((size_t)run.slot * p.heads + h) * D * D;
+  float st[WKV_KPT], u[WKV_KPT];
+#pragma unroll
+  for (int i = 0; i < WKV_KPT; ++i) {
+    const int k = k0 + i;
+    u[i] = k < D ? p.u[hc + k] : 0.f;
+    st[i] = run.start > 0 && k < D && col_ok ? S[(size_t)k * D + col] : 0.f;
+  }
+  // padding keys and columns stay zero in both tiles
+  for (int i = tid; i < 2 * WKV_TILE * ROW; i += WKV_SCAN_THREADS) scan_s[i] = 0.f;
+  __syncthreads();
+  const bool vec = !((D | hc | p.stride | p.off | p.decay_stride) & 3);  // 16-byte pieces possible
+  auto fetch = [&](int tile) {
+    float* dst = scan_s + (size_t)(tile & 1) * WKV_TILE * ROW;
+    const int first = tile * WKV_TILE, n = min(WKV_TILE, run.len - first);
+    if (n <= 0) return;
+    const int per = vec ? D / 4 : D;
+    for (int i = tid; i < n * 3 * per; i += WKV_SCAN_THREADS) {
+      const int t = i / (3 * per), e = i - t * 3 * per, which = e / per, c = e - which * per;
+      const size_t row = (size_t)(run.row0 + first + t);
+      const float* src = which == 2 ? p.decay + row * p.decay_stride + hc : p.rkv + row * p.stride + which * p.off + hc;
+      float* d = dst + t * ROW + which * DP;
+      if (vec) pfa_cp16(d + 4 * c, src + 4 * c);
+      else d[c] = src[c];
+    }
+    for (int i = tid; i < n * COLS; i += WKV_SCAN_THREADS) {
+      const int t = i / COLS, c = i - t * COLS;
+      if (blockIdx.x * COLS + c < D) dst[t * ROW + 3 * DP + c] = p.rkv[(size_t)(run.row0 + first + t) * p.stride + 2 * p.off + hc + blockIdx.x * COLS + c];
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  const int tiles = (run.len + WKV_TILE - 1) / WKV_TILE;
+  fetch(0);
+  for (int tile = 0; tile < tiles; ++tile) {
+    pfa_cp_wait_all();
+    __syncthreads();  // the tile has landed for everyone, and everyone has left the other buffer
+    fetch(tile + 1);
+    const float* base = scan_s + (size_t)(tile & 1) * WKV_TILE * ROW;
+    const int n = min(WKV_TILE, run.len - tile * WKV_TILE);
+    float mine = 0.f;  // outputs are written L tokens at a time, one per lane of the column
+#pragma unroll 4
+    for (int t = 0; t < n; ++t) {
+      const float* row = base + t * ROW;
+      const float4 r0 = *reinterpret_cast<const float4*>(row + k0), r1 = *reinterpret_cast<const float4*>(row + k0 + 4);
+      const float4 a0 = *reinterpret_cast<const float4*>(row + DP + k0), a1 = *reinterpret_cast<const float4*>(row + DP + k0 + 4);
+      const float4 w0 = *reinterpret_cast<const float4*>(row + 2 * DP + k0), w1 = *reinterpret_cast<const float4*>(row + 2 * DP + k0 + 4);
+      const float v = row[3 * DP + tid / L];
+      const float r[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
+      const float k[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+      const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+      float o = 0.f;
+#pragma unroll
+      for (int i = 0; i < WKV_KPT; ++i) {
+        const float kv = k[i] * v;
+        o = fmaf(r[i], fmaf(u[i], kv, st[i]), o);
+        st[i] = fmaf(w[i], st[i], kv);
+      }
+#pragma unroll
+      for (int s = L / 2; s > 0; s >>= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
+      if (t % L == ln) mine = o;
+      if ((t % L == L - 1 || t == n - 1) && col_ok && ln <= t % L)
+        p.o[(size_t)(run.row0 + tile * WKV_TILE + t - t % L + ln) * p.o_stride + hc + col] = mine;
+    }
+  }
+  if (col_ok)
+#pragma unroll
+    for (int i = 0; i < WKV_KPT; ++i)
+      if (k0 + i < D) S[(size_t)(k0 + i) * D + col] = st[i];
+  if (blockIdx.x == 0) {  // the heads' first blocks share the copy of the last token's h
+    const float* src = p.h + (size_t)(run.row0 + run.len - 1) * p.h_stride;
+    float* dst = p.shift + ((size_t)run.slot * 2 + ((run.start + run.len) & 1)) * p.shift_stride;
+    for (int i = h * WKV_SCAN_THREADS + tid; i < p.W; i += p.heads * WKV_SCAN_THREADS) dst[i] = src[i];
+  }
+}
+
+}  // namespace b200
