@@ -7,6 +7,12 @@ A step is one decode step (one new token for every sequence of the batch). The d
 the Llama-2-7B-shaped Q4_K_M-style model at batch 1 with a 1024-token prompt and an INT8 KV cache.
 Weights are synthetic (seeded N(0, 0.02), quantized by the package's writer); prompts are seeded
 uniform token ids. One JSON line is printed by rank 0.
+
+  python bench.py --block-model nezolix-w4096 [--steps K] [--warmup W]
+
+measures a block model instead (random bfloat16 weights in the sizes of a real model's layers): prompt ingestion and
+decode throughput, and every kind of launch alone, beside a packed-weight Llama model of the same width, feed-forward
+size, heads, layers and vocabulary.
 """
 import argparse
 import json
@@ -230,6 +236,135 @@ def parity_in_run(eng, shape, scheme, kv):
             "logit_gate_note": None if not tag.endswith("i8") else "INT8 cache: 2e-2 or a quarter of the oracle's own INT8-vs-FP32 drift (rounding flips of cached values)"}
 
 
+def block_kinds(shape, batch, rows, chunk, context, act_bytes=4):
+    """FLOPs of each timed kind of a block model's launch (selector -> name, FLOPs per launch)."""
+    s = shape
+    H, D, R, V, W = s["heads"], s["dim"], s["rot_dim"], s["vdim"], s["width"]
+    T = chunk if rows else batch
+    win = min(s["window"], context)
+    ctx = min(s["window"] - 1, context - chunk) + chunk
+    hd = s["wkv_heads"] * s["wkv_dim"]
+    kinds = {0: ("gate_up", 2 * 2 * s["ff"] * W * T), 1: ("latent_in (W_dq, W_dkv, gate)", 2 * (s["q_rank"] + s["kv_rank"] + R + H * V) * W * T),
+             2: ("o_proj", 2 * W * H * V * T), 3: ("down_proj", 2 * W * s["ff"] * T), 5: ("latent_uq", 2 * H * (D + R) * s["q_rank"] * T),
+             6: ("latent_attention", 2 * H * T * win * (D + R + V) if rows else 2 * H * T * (win * (2 * s["kv_rank"] + R) + (D + V) * s["kv_rank"])),
+             7: ("wkv_in (r, k, v, gate, w1)", 2 * (4 * hd + s["decay_rank"]) * W * T), 8: ("wkv_recurrence", 7 * hd * s["wkv_dim"] * T)}
+    if rows:
+        kinds.update({9: ("latent_expand (W_uk, W_uv)", 2 * H * (D + V) * s["kv_rank"] * ctx), 10: ("latent_append", 0), 11: ("norm_rows", 0)})
+    else:
+        kinds[4] = ("lm_head", 2 * s["vocab"] * W * T)
+    return kinds
+
+
+def run_block(args):
+    """Prompt and decode throughput of a block model and of the packed-weight model of equal size, one JSON line."""
+    pkg = __graft_entry__.load_package()
+    json_fd = os.dup(1)
+    os.dup2(2, 1)
+    shape = pkg.synth.BLOCK_SHAPES[args.block_model]
+    base = "/dev/shm" if os.path.isdir("/dev/shm") and os.access("/dev/shm", os.W_OK) else "/tmp"
+    folder = os.path.join(base, f"b200_synth_{args.block_model}")
+    if not os.path.exists(os.path.join(folder, "done")):
+        pkg.synth.write_block_model(folder, args.block_model)
+        open(os.path.join(folder, "done"), "w").close()
+    like = dict(hidden=shape["width"], ffn=shape["ff"], n_heads=shape["heads"], n_kv_heads=shape["heads"], n_layers=shape["n_layers"], vocab=shape["vocab"],
+                max_pos=8192, theta=10000.0)
+    gguf = os.path.join(base, f"b200_synth_like_{args.block_model}.gguf")
+    if not os.path.exists(gguf):
+        pkg.synth.write_gguf(gguf + ".tmp", like, scheme=0)
+        os.replace(gguf + ".tmp", gguf)
+    progress("model files ready")
+    peak, peak_tf, peak_src = peaks()
+    steps, warmup, prompt_len, chunk = args.steps or 128, max(args.warmup, 3), 4096, 1024
+    batches = (1, 8, 16, 64)
+    rng = np.random.Generator(np.random.PCG64(4321))
+    sampler = ClockSampler(0)
+    sampler.start()
+
+    def throughput(load, kv_note):
+        out = {"weights": kv_note, "decode": {}, "prompt": {}}
+        for b in batches:
+            eng = load(b, prompt_len + 2 * warmup + 2 * steps + 8 if b == 1 else 1024 + 2 * warmup + steps + 8)
+            n = prompt_len if b == 1 else 1024
+            prompts_b = [rng.integers(0, shape["vocab"], n).astype(np.int32) for _ in range(b)]
+            first = []
+            for i, p in enumerate(prompts_b):
+                eng.prefill(p[:16], slot=i)
+                eng.kv_reset(i)
+            if b == 1:
+                for m in (128, 1024, 4096):
+                    best = 1e9
+                    for _ in range(4):
+                        t0 = time.perf_counter()
+                        eng.prefill(prompts_b[0][:m], slot=0)
+                        best = min(best, time.perf_counter() - t0)
+                    out["prompt"][f"{m} tokens"] = {"tokens_per_s": round(m / best), "ms": round(best * 1e3, 3)}
+            first = eng.prefill_batch(prompts_b).argmax(axis=1)
+            _, _ = eng.generate_greedy(first, [n] * b, warmup)
+            _, ms = eng.generate_greedy(first, [n + warmup] * b, steps)
+            st = eng.stats()
+            ctx = n + warmup + steps / 2
+            reads = st["weight_bytes"] + b * st["kv_bytes_per_position"] * (min(ctx, shape["window"]) if "bf16" in kv_note else ctx)
+            t0 = time.perf_counter()
+            toks = first
+            e2e = max(1, min(steps, 64, warmup))
+            for i in range(e2e):
+                logits, _ = eng.decode(toks, [n + warmup + steps + i] * b, want_argmax=False)
+                toks = logits.argmax(axis=1).astype(np.int32)
+            dt = time.perf_counter() - t0
+            gbs = reads / (ms / steps) / 1e6
+            out["decode"][f"batch {b}"] = {"tokens_per_s": round(b * steps / ms * 1e3, 1), "ms_per_step": round(ms / steps, 4), "step_bytes": int(reads),
+                                           "GBps": round(gbs, 1), "frac_of_measured_copy": round(gbs / peak, 4), "e2e_tokens_per_s": round(b * e2e / dt, 1),
+                                           "launches_per_step": st["launches_per_step"]}
+            eng.close()
+        return out
+
+    def frac(us, nbytes, flops, fp32=False):
+        """Achieved over the slower of the two rooflines (measured copy rate; measured bf16 rate, or FP32 FMA peak 74 TFLOP/s nominal)."""
+        t_mem, t_math = nbytes / (peak * 1e3), flops / ((74.0 if fp32 else peak_tf) * 1e6)
+        return {"us": round(us, 2), "bytes": int(nbytes), "GFLOP": round(flops / 1e9, 3), "bound": "hbm" if t_mem >= t_math else "math",
+                "frac": round(max(t_mem, t_math) / us, 4)}
+
+    def block(b, ctx):
+        return pkg.Engine.from_model(folder, max_seqs=b, max_ctx=ctx)
+
+    def packed(b, ctx):
+        return pkg.Engine.from_gguf(gguf, kv_dtype=pkg.KV_I8, max_seqs=b, max_ctx=ctx)
+
+    result = {"block model": throughput(block, "bf16, bf16 latent cache, window %d" % shape["window"]), "packed model": throughput(packed, "Q8_0, INT8 KV cache")}
+    progress("throughput done")
+    kernels = {}
+    for label, b, rows in (("decode batch 1", 1, False), ("decode batch 8", 8, False), (f"prompt chunk of {chunk}", 1, True)):
+        eng = block(b, 4096)
+        kernels[label] = {}
+        for which, (name, flops) in block_kinds(shape, b, rows, chunk, 4096).items():
+            us, nbytes = eng.time_kernel(which + (16 if rows else 0), 48)
+            kernels[label][name] = frac(us, nbytes, flops, fp32=which == 8 or (which == 6 and not rows))
+        eng.close()
+    for label, b, rows in (("packed: decode batch 1", 1, False), ("packed: prompt chunk of 512", 512, True)):
+        eng = packed(b, 4096 if b == 1 else 16)
+        names = {0: "gate_up", 1: "qkv", 2: "o_proj", 3: "down_proj"}
+        T, W, F = (512 if rows else 1), like["hidden"], like["ffn"]
+        fl = {0: 4 * F * W * T, 1: 6 * W * W * T, 2: 2 * W * W * T, 3: 2 * W * F * T}
+        kernels[label] = {}
+        for which, name in names.items():
+            us, nbytes = eng.time_kernel(which + (16 if rows else 0), 48)
+            kernels[label][name] = frac(us, nbytes, fl[which])
+        eng.close()
+    eng = packed(1, 1024)
+    us, nbytes = eng.time_kernel(5, 48)
+    kernels["packed: decode batch 1"]["attention, 1024 keys"] = frac(us, nbytes, 4 * 1024 * like["hidden"], fp32=True)
+    us, nbytes = eng.time_kernel(21, 48)
+    kernels["packed: prompt chunk of 512"]["attention, 512 queries, 1024 keys"] = frac(us, nbytes, 4 * 512 * 768 * like["hidden"])
+    eng.close()
+    clocks = sampler.finish()
+    line = {"metric": f"decode tokens/s of {args.block_model}, batch 1", "value": result["block model"]["decode"]["batch 1"]["tokens_per_s"], "unit": "tokens/s",
+            "n_gpus": 1, "steps": steps, "warmup": warmup, "ms_per_step": result["block model"]["decode"]["batch 1"]["ms_per_step"], "higher_is_better": True,
+            "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "config": dict(shape, model=args.block_model, packed_like=like,
+            l2="weights read per step exceed the 126 MB L2", timing="CUDA events around the device loop / the launches; prompts by the host clock around a synchronous call"),
+            "throughput": result, "kernels": kernels, "peaks": {"hbm_GBps": peak, "bf16_TFLOPs": peak_tf, "source": peak_src}, "clocks": clocks}
+    os.write(json_fd, (json.dumps(line) + "\n").encode())
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -240,7 +375,10 @@ def main():
     ap.add_argument("--planes", type=int, default=3, choices=[2, 3])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-check", action="store_true", help="skip the in-run parity check against the golden fixtures")
+    ap.add_argument("--block-model", default=None, choices=["nezolix-w2048", "nezolix-w4096"], help="measure a block model instead of a workload")
     args = ap.parse_args()
+    if args.block_model:
+        return run_block(args)
     shape, scheme, batch, prompt_len, kv = WORKLOADS[args.workload]
     if args.steps is None:
         args.steps = 96 if shape == "llama2-70b" else 256

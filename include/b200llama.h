@@ -213,8 +213,11 @@ int b200_attention_decode_noalloc(const float* d_q, const float* d_kv_new, void*
 /* Timing and counters for the benchmark harness. */
 int b200_engine_stats(const b200_engine* e, int64_t* kernel_launches_per_step, int64_t* weight_bytes,
                       int64_t* kv_bytes_per_position);
-/* Repeats one kernel of the decode step alone (0 = the largest GEMV of a layer) `iters` times over
- * distinct layers' weights and returns its mean CUDA-event duration and algorithmic bytes. */
+/* Repeats one kernel of the decode step (or, with 16 added to the selector, of the batch / prompt path) alone `iters` times over
+ * distinct layers' weights and returns its mean CUDA-event duration and algorithmic bytes. 0 = gate/up, 1 = first projections,
+ * 2 = O projection, 3 = down projection, 4 = lm_head, 5 = attention; block models: 5 = query projection, 6 = latent attention,
+ * 7 = WKV projections, 8 = WKV recurrence, and of a prompt chunk also 9 = key / value expansion, 10 = cache append, 11 = row norm
+ * (their slots are cleared afterwards). */
 int b200_engine_time_kernel(b200_engine* e, int which, int iters, float* mean_us, int64_t* bytes_per_launch);
 
 /* Step trace (no counterpart in the reference, which has no timers besides total wall time, api.cpp:825-831).

@@ -1,5 +1,6 @@
 """Plain, slow numpy statement of the layer mechanisms of the block models (one function per mechanism): the oracle of
-the tests. Shares no code with the package. Everything is computed in float64 unless a caller passes other arrays."""
+the tests. Shares no code with the package. Everything is computed in float64; `rnd` is applied to what enters a matrix product
+(identity, or rounding to bfloat16 to learn how far that alone moves the results)."""
 import json
 import math
 import struct
@@ -46,6 +47,14 @@ def read_model(folder):
 
 
 # ---- small pieces ------------------------------------------------------------------------------------------------
+def exact(a):
+    return a
+
+
+def to_bf16(a):
+    return bf16_round(np.asarray(a, np.float32)).astype(np.float64)
+
+
 def rms(x, w, eps):
     return x / np.sqrt(np.mean(x * x, axis=-1, keepdims=True) + eps) * w
 
@@ -89,21 +98,22 @@ def rotate(x, positions, rot):
 
 
 # ---- mixers ------------------------------------------------------------------------------------------------------
-def latent_attention(h, W, m, eps, start=0, cache=None):
+def latent_attention(h, W, m, eps, start=0, cache=None, rnd=exact):
     """h [T][width] at positions start..; W(name) gives the mixer's tensors. cache: (latents, rotated keys) of the
     positions before `start`. Returns (output, new cache)."""
     T, H, D, R, VD = len(h), m["heads"], m["dim"], m["rot_dim"], m["vdim"]
     pos = np.arange(start, start + T)
-    q = (rms(h @ W("dq").T, W("dq.norm"), eps) @ W("uq").T).reshape(T, H, D + R)
-    qn, qr = q[..., :D], rotate(q[..., D:], pos, m["rot"])
+    h = rnd(h)
+    q = (rnd(rms(h @ W("dq").T, W("dq.norm"), eps)) @ W("uq").T).reshape(T, H, D + R)
+    qn, qr = rnd(q[..., :D]), rnd(rotate(q[..., D:], pos, m["rot"]))
     low = h @ W("dkv").T
-    c = rms(low[:, :m["kv_rank"]], W("dkv.norm"), eps)
-    kr = rotate(low[:, m["kv_rank"]:], pos, m["rot"])
+    c = rnd(rms(low[:, :m["kv_rank"]], W("dkv.norm"), eps))
+    kr = rnd(rotate(low[:, m["kv_rank"]:], pos, m["rot"]))
     if cache is not None:
         c, kr = np.concatenate([cache[0], c]), np.concatenate([cache[1], kr])
     N = len(c)
-    kn = (c @ W("uk").T).reshape(N, H, D)
-    v = (c @ W("uv").T).reshape(N, H, VD)
+    kn = rnd(c @ W("uk").T).reshape(N, H, D)
+    v = rnd(c @ W("uv").T).reshape(N, H, VD)
     out = np.empty((T, H, VD))
     window = (m.get("mask") or {}).get("size")
     for t in range(T):
@@ -112,9 +122,9 @@ def latent_attention(h, W, m, eps, start=0, cache=None):
         s = (np.einsum("hd,jhd->hj", qn[t], kn[lo:p + 1]) + qr[t] @ kr[lo:p + 1].T) * m["scale"]
         e = np.exp(s - s.max(axis=1, keepdims=True))
         e /= e.sum(axis=1, keepdims=True)
-        out[t] = np.einsum("hj,jhv->hv", e, v[lo:p + 1])
+        out[t] = np.einsum("hj,jhv->hv", rnd(e), v[lo:p + 1])
     o = out.reshape(T, H * VD) * sigmoid(h @ W("g").T)
-    return o @ W("o").T, (c, kr)
+    return rnd(o) @ W("o").T, (c, kr)
 
 
 def wkv_recurrence(r, k, v, w, u, S):
@@ -128,22 +138,23 @@ def wkv_recurrence(r, k, v, w, u, S):
     return out, S
 
 
-def wkv(h, W, m, eps, state=None):
+def wkv(h, W, m, eps, state=None, rnd=exact):
     """state: (last h, S). Returns (output, new state)."""
     T, H, D = len(h), m["heads"], m["dim"]
     last, S = state if state is not None else (np.zeros(h.shape[1]), np.zeros((H, D, D)))
     prev = np.concatenate([last[None], h[:-1]])
-    mix = {s: h + (prev - h) * W("mu." + s) for s in "rkvgw"}
+    mix = {s: rnd(h + (prev - h) * W("mu." + s)) for s in "rkvgw"}
     r, k, v = ((mix[s] @ W(s).T).reshape(T, H, D) for s in "rkv")
     gate = silu(mix["g"] @ W("g").T)
-    w = np.exp(-np.exp(np.tanh(mix["w"] @ W("w1").T) @ W("w2").T + W("w0"))).reshape(T, H, D)
+    w = np.exp(-np.exp(rnd(np.tanh(mix["w"] @ W("w1").T)) @ W("w2").T + W("w0"))).reshape(T, H, D)
     o, S = wkv_recurrence(r, k, v, w, W("u"), S)
     o = o / np.sqrt(np.mean(o * o, axis=-1, keepdims=True) + eps)
-    return (o.reshape(T, H * D) * W("norm") * gate) @ W("o").T, (h[-1], S)
+    return rnd(o.reshape(T, H * D) * W("norm") * gate) @ W("o").T, (h[-1], S)
 
 
-def dense_relu(h, W):
-    return (np.maximum(h @ W("gate").T, 0) * (h @ W("up").T)) @ W("down").T
+def dense_relu(h, W, rnd=exact):
+    h = rnd(h)
+    return rnd(np.maximum(h @ W("gate").T, 0) * (h @ W("up").T)) @ W("down").T
 
 
 # ---- model -------------------------------------------------------------------------------------------------------
@@ -156,7 +167,8 @@ def layer_runs(cfg):
 
 
 class PlainModel:
-    def __init__(self, cfg, tensors):
+    def __init__(self, cfg, tensors, rnd=exact):
+        self.rnd = rnd
         self.cfg, self.t = cfg, {k: np.asarray(v, np.float64) for k, v in tensors.items()}
         self.reset()
 
@@ -173,17 +185,17 @@ class PlainModel:
             W = lambda s: self.t[f"l{l}.mix.{s}"]
             h = rms(x, N("norm1"), eps)
             if lay["type"] == "wkv":
-                y, self.state[i] = wkv(h, W, lay["mixer"], eps, self.state[i])
+                y, self.state[i] = wkv(h, W, lay["mixer"], eps, self.state[i], self.rnd)
             else:
-                y, self.state[i] = latent_attention(h, W, lay["mixer"], eps, self.pos, self.state[i])
+                y, self.state[i] = latent_attention(h, W, lay["mixer"], eps, self.pos, self.state[i], self.rnd)
             x = x + rms(y, N("norm1b"), eps)
             if lay.get("mlp"):
-                y = dense_relu(rms(x, N("norm2"), eps), lambda s: self.t[f"l{l}.mlp.{s}"])
+                y = dense_relu(rms(x, N("norm2"), eps), lambda s: self.t[f"l{l}.mlp.{s}"], self.rnd)
                 x = x + rms(y, N("norm2b"), eps)
             if trace is not None:
                 trace.append(x.copy())
         self.pos += len(x)
-        return rms(x, self.t["final.norm"], eps) @ self.t["head"].T
+        return self.rnd(rms(x, self.t["final.norm"], eps)) @ self.t["head"].T
 
 
 def greedy(cfg, tensors, prompt, steps):

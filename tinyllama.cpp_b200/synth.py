@@ -1,7 +1,9 @@
 """Synthetic models: named shapes from the benchmark configurations and a ctypes front end to the
 GGUF writer / quantizers in csrc/synth.cpp."""
 import ctypes
+import json
 import os
+import struct
 
 import numpy as np
 
@@ -77,3 +79,85 @@ def quantize(ggml_type, x):
     if rc:
         raise RuntimeError(f"b200_synth_quantize failed with status {rc}")
     return out
+
+
+# Block models of a real model's layer sizes: three latent-attention layers, then one WKV layer, repeated.
+BLOCK_SHAPES = {
+    "nezolix-w2048": dict(width=2048, ff=5632, vocab=32000, n_layers=8, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=256,
+                          window=1024, wkv_heads=32, wkv_dim=64, decay_rank=64),
+    "nezolix-w4096": dict(width=4096, ff=11008, vocab=32000, n_layers=8, heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512,
+                          window=1024, wkv_heads=64, wkv_dim=64, decay_rank=64),
+}
+
+
+def block_config(shape):
+    s = BLOCK_SHAPES[shape] if isinstance(shape, str) else shape
+    attn = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": s["ff"]},
+            "mixer": {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot_dim"], "vdim": s["vdim"], "q_rank": s["q_rank"], "kv_rank": s["kv_rank"],
+                      "scale": (s["dim"] + s["rot_dim"]) ** -0.5, "mask": {"size": s["window"]},
+                      "rot": {"base": 10000.0, "dims": s["rot_dim"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    wkv = {"type": "wkv", "mlp": {"kind": "dense", "ff": s["ff"]}, "mixer": {"heads": s["wkv_heads"], "dim": s["wkv_dim"]}}
+    return {"architecture": "Nezolix", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "loop": None,
+            "layers": [wkv if l % 4 == 3 else attn for l in range(s["n_layers"])]}
+
+
+def block_tensors(cfg, decay_rank):
+    """(name, shape) of every tensor of a block model."""
+    W = cfg["width"]
+    out = [("embed", (cfg["vocab"], W))]
+    for i, l in enumerate(cfg["layers"]):
+        L, m = f"l{i}.", l["mixer"]
+        H, D = m["heads"], m["dim"]
+        out += [(L + "norm1", (W,)), (L + "norm1b", (W,))]
+        if l["type"] == "latent_attention":
+            out += [(L + "mix." + n, s) for n, s in (
+                ("dq", (m["q_rank"], W)), ("dq.norm", (m["q_rank"],)), ("uq", (H * (D + m["rot_dim"]), m["q_rank"])), ("dkv", (m["kv_rank"] + m["rot_dim"], W)),
+                ("dkv.norm", (m["kv_rank"],)), ("uk", (H * D, m["kv_rank"])), ("uv", (H * m["vdim"], m["kv_rank"])), ("g", (H * m["vdim"], W)), ("o", (W, H * m["vdim"])))]
+        else:
+            out += [(L + "mix.mu." + n, (W,)) for n in "rkvgw"] + [(L + "mix." + n, (H * D, W)) for n in "rkvg"]
+            out += [(L + "mix." + n, s) for n, s in (("w1", (decay_rank, W)), ("w2", (H * D, decay_rank)), ("w0", (H * D,)), ("u", (H, D)), ("norm", (H * D,)), ("o", (W, H * D)))]
+        if l["mlp"]:
+            ff = l["mlp"]["ff"]
+            out += [(L + "norm2", (W,)), (L + "norm2b", (W,)), (L + "mlp.gate", (ff, W)), (L + "mlp.up", (ff, W)), (L + "mlp.down", (W, ff))]
+    return out + [("final.norm", (W,)), ("head", (cfg["vocab"], W))]
+
+
+def write_block_model(folder, shape, seed=1234, sigma=0.02):
+    """Writes config.json and model.safetensors of a BLOCK_SHAPES entry: N(0, sigma) matrices (slices of one seeded block of
+    16 Mi values at seeded offsets), unit norms, token-shift mixes in [0, 1), decay biases around -3."""
+    os.makedirs(folder, exist_ok=True)
+    s = BLOCK_SHAPES[shape] if isinstance(shape, str) else shape
+    cfg = block_config(shape)
+    with open(os.path.join(folder, "config.json"), "w") as f:
+        json.dump(cfg, f)
+    names = block_tensors(cfg, s["decay_rank"])
+    head, at = {}, 0
+    for name, shp in names:
+        n = int(np.prod(shp)) * 2
+        head[name] = {"dtype": "BF16", "shape": list(shp), "data_offsets": [at, at + n]}
+        at += n
+    rng = np.random.default_rng(seed)
+    block = rng.standard_normal(1 << 24, dtype=np.float32) * sigma
+    block = (block.view(np.uint32) >> 16).astype(np.uint16)
+
+    def bits(a):
+        return (np.ascontiguousarray(a, np.float32).view(np.uint32) >> 16).astype(np.uint16)
+
+    h = json.dumps(head).encode()
+    with open(os.path.join(folder, "model.safetensors"), "wb") as f:
+        f.write(struct.pack("<Q", len(h)) + h)
+        for name, shp in names:
+            n = int(np.prod(shp))
+            if "norm" in name:
+                f.write(bits(np.ones(n)).tobytes())
+            elif ".mu." in name:
+                f.write(bits(rng.uniform(0, 1, n)).tobytes())
+            elif name.endswith(".w0"):
+                f.write(bits(rng.normal(-3, 1, n)).tobytes())
+            else:
+                while n:
+                    o = int(rng.integers(0, block.size))
+                    k = min(n, block.size - o)
+                    f.write(block[o:o + k].tobytes())
+                    n -= k
+    return folder
