@@ -55,6 +55,7 @@ struct BlockModel {
   int cat_stride = 0, q_stride = 0, att_stride = 0, act_stride = 0;
   float *part_o = nullptr, *part_ml = nullptr;
   int* tickets = nullptr;
+  __nv_bfloat16* q_split[2] = {nullptr, nullptr};  // absorbed queries of decode attention: value and remainder, [max_seqs][heads][cache row]
   // row path: prompt chunks and batches of 16 and more, [rows_cap] rows
   float *rx = nullptr, *ry = nullptr, *rh = nullptr, *rcat = nullptr, *rq = nullptr, *rdecay = nullptr, *ro = nullptr;
   void *ra[5] = {nullptr};      // operand rows of the next matmul (five for token-shift mixes)
@@ -64,6 +65,11 @@ struct BlockModel {
   size_t meta_cap = 0;
   void *ctx = nullptr, *ctx_kr = nullptr, *ctx_kv = nullptr;  // expanded context of a chunk
   size_t ctx_cap[3] = {0, 0, 0};
+  // split-K workspace of the tensor-core matmul
+  float* gemm_ws = nullptr;
+  size_t gemm_ws_floats = 0;
+  int* gemm_tickets = nullptr;
+  int gemm_tickets_cap = 0;
   float* logits = nullptr;      // [rows][vocab] of the wanted places, grown on demand
   size_t logits_cap = 0;
 };

@@ -1,13 +1,14 @@
 // Matmul over bfloat16 weights for prompts and batches of 16 and more of the block models:
 //   Y[t][row] = act(sum_k W[row][k] * X[t][k])      (W and X bfloat16, FP32 accumulation)
 //
-// dense_gemm_kernel: 5th-generation tensor cores. Weight rows are the MMA's M side (128 per CTA tile), tokens its N
-// side (32 to 256 per tile). A producer lane moves both operands' 64-element K slices with TMA
+// dense_gemm_kernel: 5th-generation tensor cores, one persistent CTA per SM. Weight rows are the MMA's M side (128 per
+// tile), tokens its N side (32 to 256 per tile). A producer lane moves both operands' 64-element K slices with TMA
 // (cp.async.bulk.tensor.2d, 128-byte swizzle; rows, tokens and elements beyond the matrices read as zero, so every
-// size is served), an MMA lane issues tcgen05.mma into a 128-lane x NT-column FP32 tile in tensor memory, four warps
-// read it back (tcgen05.ld) and apply the segment's activation. Two CTAs share an SM (at most 256 tensor-memory columns
-// each), so one tile's epilogue overlaps the other's products. Segments (the projections of one input) share a launch;
-// each has its own weights, activation rows and output.
+// size is served), an MMA lane issues tcgen05.mma into one of two accumulators in tensor memory, and eight warps read the
+// other one back (tcgen05.ld) and apply the segment's activation: a tile's epilogue runs under the next tile's products.
+// Token tiles of the same weight rows follow one another, so a weight row comes from HBM once. Launches with few tiles
+// (small batches) split K: partial tiles go to a workspace and the last CTA of a tile adds them in order.
+// Segments (the projections of one input) share a launch; each has its own weights, activation rows and output.
 //
 // sgemm_kernel: the same product in plain FP32 arithmetic (FFMA on FP32 activations; the bfloat16 weights are exact in
 // FP32), for engines that run in 32-bit.
@@ -17,9 +18,10 @@
 
 namespace b200 {
 
-constexpr int DGM_THREADS = 192;  // four epilogue warps, the TMA warp, the MMA warp
+constexpr int DGM_EPI_WARPS = 8;
+constexpr int DGM_THREADS = 32 * DGM_EPI_WARPS + 64;  // + the TMA warp and the MMA warp
 constexpr int DGM_MAX_STAGES = 8;
-constexpr int DGM_SMEM_PER_CTA = 110 * 1024;  // two CTAs per SM
+constexpr int DGM_SMEM = 216 * 1024;
 
 struct DgmSeg {
   const __nv_bfloat16* w;  // [rows][pad8(K)]
@@ -37,7 +39,11 @@ struct DgmSeg {
 struct DgmParams {
   DgmSeg seg[DGV_MAX_SEGS];
   int nseg, K, T;
-  int NT, stages, tmem_cols;
+  int NT, stages, acc_cols;    // token tile, ring depth, tensor-memory columns per accumulator
+  int tiles_m, tiles_n;        // 128-row tiles over all segments, token tiles
+  int ksplit, ksteps;          // K splits and 64-element steps per split
+  float* ws;                   // split K: partial tiles [ksplit][tile][NT][128]
+  int* tickets;                // split K: one per tile, zero between launches
   int* error_flag;
 };
 
@@ -46,104 +52,226 @@ struct alignas(64) DgmMaps {
 };
 
 struct DgmShared {
-  unsigned long long full[DGM_MAX_STAGES], empty[DGM_MAX_STAGES], done;
+  unsigned long long full[DGM_MAX_STAGES], empty[DGM_MAX_STAGES], acc_full[2], acc_empty[2];
   uint32_t tmem_base;
-  int abort_flag, issued;  // steps whose copies have been issued
+  int abort_flag, issued;  // issued: K slices whose copies have been requested
+  int last;
 };
 
 // kind::f16 with bfloat16 operands: D = F32, A and B = BF16 and K-major
 __host__ __device__ __forceinline__ uint32_t dgm_idesc(int n) { return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(TC_M >> 4) << 24); }
 
-__device__ __forceinline__ void dgm_fail(const DgmParams& p, DgmShared* sh) {
+__device__ __forceinline__ bool dgm_wait(const DgmParams& p, DgmShared* sh, void* bar, uint32_t parity) {
+  if (*(volatile int*)&sh->abort_flag) return false;
+  if (mbar_wait(bar, parity)) return true;
   *(volatile int*)&sh->abort_flag = 1;
   if (p.error_flag) *reinterpret_cast<volatile int*>(p.error_flag) = 1;
+  return false;
 }
 
-__device__ __forceinline__ void dgm_store(const DgmSeg& sg, int t, int row, float v) {
-  if (sg.y_bf16) static_cast<__nv_bfloat16*>(sg.y)[(size_t)t * sg.y_stride + row] = __float2bfloat16(v);
-  else static_cast<float*>(sg.y)[(size_t)t * sg.y_stride + row] = v;
+// this warp's 32 TMEM lanes, 16 consecutive columns
+__device__ __forceinline__ void tc_ld16(uint32_t taddr, float (&v)[16]) {
+  uint32_t r[16];
+  asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]),
+                 "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
+               : "r"(taddr));
+  asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+  for (int i = 0; i < 16; ++i) v[i] = __uint_as_float(r[i]);
+}
+
+__device__ __forceinline__ void dgm_put(float* y, float v) { *y = v; }
+__device__ __forceinline__ void dgm_put(__nv_bfloat16* y, float v) { *y = __float2bfloat16(v); }
+
+// Sixteen columns (tokens t0 ..) of this lane's row: activation and store. ACT is a compile-time copy of sg.act.
+template <int ACT, typename Y>
+__device__ __forceinline__ void dgm_store16(const DgmSeg& sg, int row, int t0, int T, float aux, const float (&v)[16]) {
+  if (ACT == ACT_RELU_GLU) {
+    const int o = (row >> 4) * 8 + (row & 7);
+    const bool mine = !(row & 8) && o < sg.outs;
+    Y* y = static_cast<Y*>(sg.y) + (size_t)t0 * sg.y_stride + o;
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      const float up = __shfl_sync(0xffffffffu, v[j], ((threadIdx.x & 31) & 23) + 8);
+      if (mine && t0 + j < T) dgm_put(y, fmaxf(v[j], 0.f) * up);
+      y += sg.y_stride;
+    }
+  } else if (row < sg.rows) {
+    Y* y = static_cast<Y*>(sg.y) + (size_t)t0 * sg.y_stride + row;
+    const int n = min(16, T - t0);
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      if (j < n) dgm_put(y, dense_act(ACT, v[j], aux));
+      y += sg.y_stride;
+    }
+  }
+}
+template <typename Y>
+__device__ __forceinline__ void dgm_store16(const DgmSeg& sg, int row, int t0, int T, float aux, const float (&v)[16]) {
+  switch (sg.act) {
+    case ACT_SIGMOID: dgm_store16<ACT_SIGMOID, Y>(sg, row, t0, T, aux, v); break;
+    case ACT_SILU: dgm_store16<ACT_SILU, Y>(sg, row, t0, T, aux, v); break;
+    case ACT_TANH: dgm_store16<ACT_TANH, Y>(sg, row, t0, T, aux, v); break;
+    case ACT_DECAY: dgm_store16<ACT_DECAY, Y>(sg, row, t0, T, aux, v); break;
+    case ACT_RELU_GLU: dgm_store16<ACT_RELU_GLU, Y>(sg, row, t0, T, aux, v); break;
+    default: dgm_store16<ACT_NONE, Y>(sg, row, t0, T, aux, v);
+  }
 }
 
 __host__ __device__ __forceinline__ size_t dgm_stage_bytes(int NT) { return (size_t)TC_M * 128 + (size_t)NT * 128; }
 
-// grid = (128-row tiles over all segments, token tiles)
-__global__ void __launch_bounds__(DGM_THREADS, 2) dense_gemm_kernel(const DgmParams p, const __grid_constant__ DgmMaps maps) {
+// One unit of work: a tile of 128 rows x NT tokens over a range of K.
+struct DgmUnit {
+  int seg, row0, t0, tile, k0, steps;
+};
+__device__ __forceinline__ DgmUnit dgm_unit(const DgmParams& p, int u) {
+  DgmUnit r;
+  const int n = u % p.tiles_n, rest = u / p.tiles_n, kz = rest % p.ksplit;
+  int m = rest / p.ksplit;
+  r.tile = m * p.tiles_n + n;
+  r.seg = 0;
+  while (r.seg + 1 < p.nseg && m >= (p.seg[r.seg].rows + TC_M - 1) / TC_M) { m -= (p.seg[r.seg].rows + TC_M - 1) / TC_M; ++r.seg; }
+  r.row0 = m * TC_M;
+  r.t0 = n * p.NT;
+  r.k0 = kz * p.ksteps;
+  r.steps = min(p.ksteps, (p.K + TC_KC - 1) / TC_KC - r.k0);
+  return r;
+}
+
+// grid = min(units, SMs)
+__global__ void __launch_bounds__(DGM_THREADS, 1) dense_gemm_kernel(const DgmParams p, const __grid_constant__ DgmMaps maps) {
   extern __shared__ uint8_t dgm_smem_raw[];
   __shared__ DgmShared sh;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   uint8_t* smem = reinterpret_cast<uint8_t*>(((uintptr_t)dgm_smem_raw + 1023) & ~(uintptr_t)1023);
   const uint32_t stage_bytes = (uint32_t)dgm_stage_bytes(p.NT);
-  int seg = 0, mt = blockIdx.x;
-  while (seg + 1 < p.nseg && mt >= (p.seg[seg].rows + TC_M - 1) / TC_M) { mt -= (p.seg[seg].rows + TC_M - 1) / TC_M; ++seg; }
-  const DgmSeg& sg = p.seg[seg];
-  const int row0 = mt * TC_M, t0 = blockIdx.y * p.NT;
-  const int nsteps = (p.K + TC_KC - 1) / TC_KC;
+  const int units = p.tiles_m * p.tiles_n * p.ksplit;
   if (tid == 0) {
     for (int i = 0; i < DGM_MAX_STAGES; ++i) { mbar_init(&sh.full[i], 1); mbar_init(&sh.empty[i], 1); }
-    mbar_init(&sh.done, 1);
+    for (int i = 0; i < 2; ++i) { mbar_init(&sh.acc_full[i], 1); mbar_init(&sh.acc_empty[i], DGM_EPI_WARPS); }
     sh.abort_flag = 0;
     sh.issued = 0;
     asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
   }
-  if (warp == 0) tc_alloc(&sh.tmem_base, p.tmem_cols);
+  if (warp == 0) tc_alloc(&sh.tmem_base, 2 * p.acc_cols);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_d = sh.tmem_base;
+  const uint32_t tmem = sh.tmem_base;
 
-  if (warp == 4) {
+  if (warp == DGM_EPI_WARPS) {
+    // ---- producer lane ----
     if (lane == 0) {
-      for (int s = 0; s < nsteps; ++s) {
-        const int st = s % p.stages;
-        if (s >= p.stages && !mbar_wait(&sh.empty[st], (uint32_t)((s / p.stages - 1) & 1))) { dgm_fail(p, &sh); break; }
-        uint8_t* a = smem + (size_t)st * stage_bytes;
-        mbar_expect_tx(&sh.full[st], stage_bytes);
-        tc_tma_load_2d(a, &maps.w[seg], s * TC_KC, row0, &sh.full[st]);
-        tc_tma_load_2d(a + TC_M * 128, &maps.x[seg], s * TC_KC, t0, &sh.full[st]);
-        sh.issued = s + 1;
+      int s = 0, st = 0;
+      uint32_t ph = 1;  // a fresh ring's slots count as empty
+      bool ok = true;
+      for (int u = blockIdx.x; u < units && ok; u += gridDim.x) {
+        const DgmUnit w = dgm_unit(p, u);
+        for (int k = 0; k < w.steps; ++k) {
+          if (s >= p.stages && !(ok = dgm_wait(p, &sh, &sh.empty[st], ph))) break;
+          uint8_t* a = smem + (size_t)st * stage_bytes;
+          mbar_expect_tx(&sh.full[st], stage_bytes);
+          tc_tma_load_2d(a, &maps.w[w.seg], (w.k0 + k) * TC_KC, w.row0, &sh.full[st]);
+          tc_tma_load_2d(a + TC_M * 128, &maps.x[w.seg], (w.k0 + k) * TC_KC, w.t0, &sh.full[st]);
+          sh.issued = ++s;
+          if (++st == p.stages) { st = 0; ph ^= 1u; }
+        }
       }
     }
     __syncwarp();
-  } else if (warp == 5) {
+  } else if (warp == DGM_EPI_WARPS + 1) {
+    // ---- MMA lane ----
     if (lane == 0) {
       const uint32_t idesc = dgm_idesc(p.NT);
+      int st = 0, n = 0;
+      uint32_t ph = 0;
       bool ok = true;
-      for (int s = 0; s < nsteps && ok; ++s) {
-        const int st = s % p.stages;
-        ok = mbar_wait(&sh.full[st], (uint32_t)((s / p.stages) & 1));
-        if (!ok) break;
+      for (int u = blockIdx.x; u < units && ok; u += gridDim.x, ++n) {
+        const DgmUnit w = dgm_unit(p, u);
+        const int buf = n & 1;
+        if (n >= 2 && !(ok = dgm_wait(p, &sh, &sh.acc_empty[buf], (uint32_t)((n / 2 - 1) & 1)))) break;
         tc_fence_after();
-        const uint32_t a = smem_u32(smem + (size_t)st * stage_bytes);
-        const uint64_t ad = tc_smem_desc(a), bd = tc_smem_desc(a + TC_M * 128);
+        const uint32_t d = tmem + (uint32_t)(buf * p.acc_cols);
+        for (int k = 0; k < w.steps; ++k) {
+          if (!(ok = dgm_wait(p, &sh, &sh.full[st], ph))) break;
+          tc_fence_after();
+          const uint32_t a = smem_u32(smem + (size_t)st * stage_bytes);
+          const uint64_t ad = tc_smem_desc(a), bd = tc_smem_desc(a + TC_M * 128);
 #pragma unroll
-        for (int k4 = 0; k4 < 4; ++k4) tc_mma_f16(tmem_d, ad + 2 * k4, bd + 2 * k4, idesc, (s | k4) ? 1u : 0u);
-        tc_commit(&sh.empty[st]);
+          for (int k4 = 0; k4 < 4; ++k4) tc_mma_f16(d, ad + 2 * k4, bd + 2 * k4, idesc, (k | k4) ? 1u : 0u);
+          tc_commit(&sh.empty[st]);
+          if (++st == p.stages) { st = 0; ph ^= 1u; }
+        }
+        if (ok) tc_commit(&sh.acc_full[buf]);
       }
-      if (!ok) dgm_fail(p, &sh);
-      tc_commit(&sh.done);
     }
     __syncwarp();
   } else {
-    if (!mbar_wait(&sh.done, 0u)) dgm_fail(p, &sh);
-    __syncwarp();
-    tc_fence_after();
-    if (!*(volatile int*)&sh.abort_flag) {
-      const int row = row0 + 32 * warp + lane;
+    // ---- epilogue warps: lanes 32 (w & 3) .. of the accumulator = weight rows, the two groups of four split the tokens ----
+    const int r = 32 * (warp & 3) + lane, c_begin = (warp >> 2) * (p.NT / 2), c_end = c_begin + p.NT / 2;
+    auto store = [&](const DgmSeg& sg, int row, int t0, float aux, const float (&v)[16]) {
+      if (sg.y_bf16) dgm_store16<__nv_bfloat16>(sg, row, t0, p.T, aux, v);
+      else dgm_store16<float>(sg, row, t0, p.T, aux, v);
+    };
+    int n = 0;
+    for (int u = blockIdx.x; u < units; u += gridDim.x, ++n) {
+      const DgmUnit w = dgm_unit(p, u);
+      const int buf = n & 1;
+      const uint32_t parity = (uint32_t)((n / 2) & 1);
+      if (p.ksplit > 1) {  // one decision for all epilogue warps: they meet on barriers below
+        if (tid == 0) sh.last = dgm_wait(p, &sh, &sh.acc_full[buf], parity);
+        asm volatile("bar.sync 1, %0;" ::"n"(32 * DGM_EPI_WARPS) : "memory");
+        const bool go = sh.last != 0;
+        asm volatile("bar.sync 1, %0;" ::"n"(32 * DGM_EPI_WARPS) : "memory");
+        if (!go) break;
+        mbar_wait(&sh.acc_full[buf], parity);  // complete already: orders this thread's reads
+        __syncwarp();
+      } else if (!__shfl_sync(0xffffffffu, (int)(lane == 0 ? dgm_wait(p, &sh, &sh.acc_full[buf], parity) : 0), 0)) {
+        break;  // one decision per warp: the loads below need all its lanes
+      }
+      tc_fence_after();
+      const DgmSeg& sg = p.seg[w.seg];
+      const int row = w.row0 + r;
       const float aux = sg.aux && row < sg.rows ? sg.aux[row] : 0.f;
-      for (int c0 = 0; c0 < p.NT && t0 + c0 < p.T; c0 += 8) {
-        float v[8];
-        tc_ld8(tmem_d + ((uint32_t)(32 * warp) << 16) + (uint32_t)c0, v);
+      const uint32_t base = tmem + ((uint32_t)(32 * (warp & 3)) << 16) + (uint32_t)(buf * p.acc_cols);
+      float* part = p.ws + ((size_t)((w.k0 / p.ksteps) * p.tiles_m * p.tiles_n + w.tile) * p.NT) * TC_M + r;
+      for (int c = c_begin; c < c_end && w.t0 + c < p.T; c += 16) {
+        float v[16];
+        tc_ld16(base + (uint32_t)c, v);
+        if (p.ksplit > 1) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) {
-          const int t = t0 + c0 + j;
-          if (sg.act == ACT_RELU_GLU) {
-            const float up = __shfl_sync(0xffffffffu, v[j], (lane & 23) + 8);
-            const int o = (row >> 4) * 8 + (row & 7);
-            if (!(row & 8) && o < sg.outs && t < p.T) dgm_store(sg, t, o, fmaxf(v[j], 0.f) * up);
-          } else if (row < sg.rows && t < p.T) {
-            dgm_store(sg, t, row, dense_act(sg.act, v[j], aux));
+          for (int j = 0; j < 16; ++j) part[(size_t)(c + j) * TC_M] = v[j];
+        } else {
+          store(sg, row, w.t0 + c, aux, v);
+        }
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(&sh.acc_empty[buf]);
+      if (p.ksplit > 1) {
+        __threadfence();
+        asm volatile("bar.sync 1, %0;" ::"n"(32 * DGM_EPI_WARPS) : "memory");
+        if (tid == 0) {
+          sh.last = atomicAdd(&p.tickets[w.tile], 1) == p.ksplit - 1;
+          if (sh.last) p.tickets[w.tile] = 0;
+        }
+        asm volatile("bar.sync 1, %0;" ::"n"(32 * DGM_EPI_WARPS) : "memory");
+        if (sh.last) {
+          __threadfence();
+          const size_t step = (size_t)p.tiles_m * p.tiles_n * p.NT * TC_M;
+          const float* sum = p.ws + (size_t)w.tile * p.NT * TC_M + r;
+          for (int c = c_begin; c < c_end && w.t0 + c < p.T; c += 16) {
+            float v[16];
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = 0.f;
+            for (int z = 0; z < p.ksplit; ++z)
+#pragma unroll
+              for (int j = 0; j < 16; ++j) v[j] += __ldcg(sum + z * step + (size_t)(c + j) * TC_M);
+            store(sg, row, w.t0 + c, aux, v);
           }
         }
+        asm volatile("bar.sync 1, %0;" ::"n"(32 * DGM_EPI_WARPS) : "memory");  // sh.last is read before the next unit writes it
       }
     }
   }
@@ -152,7 +280,7 @@ __global__ void __launch_bounds__(DGM_THREADS, 2) dense_gemm_kernel(const DgmPar
   // The MMA lane waits for every copy; only after a give-up may some still be in flight, and the block outlives them.
   if (sh.abort_flag && tid == 0)
     for (int s = max(0, sh.issued - p.stages); s < sh.issued; ++s) mbar_wait(&sh.full[s % p.stages], (uint32_t)((s / p.stages) & 1));
-  if (warp == 0) tc_dealloc(tmem_d, p.tmem_cols);
+  if (warp == 0) tc_dealloc(tmem, 2 * p.acc_cols);
 }
 
 // 64 rows x 64 tokens per block of 256 threads, 4 x 4 outputs per thread, K in steps of 16. grid = (row tiles over all
@@ -202,7 +330,9 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const DgmParams p) {
         const int row = r0 + 4 * tr + i, t = t0 + 4 * tt + j;
         if (glu && half == 0) { kept[i][j] = fmaxf(acc[i][j], 0.f); continue; }
         if (row >= sg.outs || t >= p.T) continue;
-        dgm_store(sg, t, row, glu ? kept[i][j] * acc[i][j] : dense_act(sg.act, acc[i][j], sg.aux ? sg.aux[row] : 0.f));
+        const float v = glu ? kept[i][j] * acc[i][j] : dense_act(sg.act, acc[i][j], sg.aux ? sg.aux[row] : 0.f);
+        if (sg.y_bf16) static_cast<__nv_bfloat16*>(sg.y)[(size_t)t * sg.y_stride + row] = __float2bfloat16(v);
+        else static_cast<float*>(sg.y)[(size_t)t * sg.y_stride + row] = v;
       }
   }
 }

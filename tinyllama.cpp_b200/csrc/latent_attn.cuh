@@ -7,9 +7,11 @@
 //                          contiguously (history from the ring, then the new ones) for the key / value expansion
 //   latent_prefill_kernel  prompts: 64 queries of one head per block over expanded keys and values, 64-key tiles, online
 //                          softmax, bfloat16 tensor-core products (mma.sync m16n8k16) with FP32 scores and sums
-//   latent_decode_kernel   one token of several sequences: works on the latents themselves. The query's unrotated part is
+//   decode                 one token of several sequences: works on the latents themselves. The query's unrotated part is
 //                          taken through W_uk once (q . W_uk c = (W_uk^T q) . c), scores and the weighted sum run over c,
-//                          and the sum is taken through W_uv at the end. FP32 arithmetic on the cached rows.
+//                          and the sum is taken through W_uv at the end. latent_decode_kernel does all of it for one
+//                          head in FP32 (32-bit engines); bfloat16 engines split it into three launches
+//                          (latent_absorb_kernel, latent_split_kernel, latent_merge_kernel)
 //
 // A = type of the cache and of matmul operands: __nv_bfloat16, or float in a 32-bit engine.
 #pragma once
@@ -339,6 +341,368 @@ __global__ void __launch_bounds__(LAD_THREADS) latent_decode_kernel(const Latent
   }
 }
 
+__device__ __forceinline__ void lap_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile(
+      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
+  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
+  return *reinterpret_cast<const uint32_t*>(&v);
+}
+
+// ---- decode on the tensor cores (bfloat16 cache) -------------------------------------------------------------------
+// Three launches: latent_absorb_kernel takes the queries through W_uk and appends the new rows, latent_split_kernel runs
+// scores and weighted sums for 16 heads and one run of keys per block, latent_merge_kernel merges the runs and goes
+// through W_uv. The cached rows are bfloat16 as they are; queries and attention weights enter the products as the sum of
+// two bfloat16 numbers (value and remainder), so that they keep 16 bits of mantissa and the scores FP32 character.
+
+__device__ __forceinline__ void split_bf16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
+  hi = __float2bfloat16(v);
+  lo = __float2bfloat16(v - __bfloat162float(hi));
+}
+
+constexpr int LAB_THREADS = 256;
+constexpr int LAB_COLS = 64;   // latent columns per block
+constexpr int LAB_BATCH = 8;   // sequences per block
+constexpr int LAB_KEEP = 8;    // pieces of W_uk a thread requests ahead (dim up to 256)
+
+struct LatentAbsorbParams {
+  LatentDecodeParams d;
+  __nv_bfloat16* q_hi;  // [batch][heads][qrow]: scaled query in the layout of a cache row, zero-filled up to qrow
+  __nv_bfloat16* q_lo;
+  int qrow, batch;
+};
+
+// grid = (kvp / 64 rounded up, heads, batch / 8 rounded up)
+__global__ void __launch_bounds__(LAB_THREADS) latent_absorb_kernel(const LatentAbsorbParams a) {
+  const LatentDecodeParams& p = a.d;
+  extern __shared__ __align__(16) float lab_s[];  // queries [LAB_BATCH][dim], then partial sums [8 warps][LAB_BATCH][64]
+  __shared__ float red[LAB_THREADS / 32];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y;
+  const int b0 = blockIdx.z * LAB_BATCH, nb = min(LAB_BATCH, a.batch - b0);
+  float* part = lab_s + LAB_BATCH * p.dim;
+  pdl_launch_dependents();
+  // thread = (8 columns, every 32nd row of the head's W_uk): pieces requested before anything else
+  const int ch = tid & 7, grp = tid >> 3, col = blockIdx.x * LAB_COLS + 8 * ch;
+  const bool col_ok = col < p.kvp;
+  const __nv_bfloat16* uk = p.uk + (size_t)h * p.dim * p.kvp;
+  uint4 w[LAB_KEEP];
+#pragma unroll
+  for (int i = 0; i < LAB_KEEP; ++i) {
+    const int d = grp + 32 * i;
+    w[i] = col_ok && d < p.dim ? ldg128(uk + (size_t)d * p.kvp + col) : make_uint4(0, 0, 0, 0);
+  }
+  pdl_wait();
+  const int qd = p.dim + p.rot_dim;
+  for (int i = tid; i < nb * p.dim; i += LAB_THREADS) {
+    const int b = i / p.dim, d = i - b * p.dim;
+    lab_s[i] = p.q[(size_t)(b0 + b) * p.q_stride + h * qd + d] * p.scale;
+  }
+  __syncthreads();
+  for (int b = 0; b < nb; ++b) {
+    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    const float* q = lab_s + b * p.dim;
+    auto add = [&](const uint4& u, float x) {
+      acc[0] = fmaf(bf_lo(u.x), x, acc[0]); acc[1] = fmaf(bf_hi(u.x), x, acc[1]); acc[2] = fmaf(bf_lo(u.y), x, acc[2]); acc[3] = fmaf(bf_hi(u.y), x, acc[3]);
+      acc[4] = fmaf(bf_lo(u.z), x, acc[4]); acc[5] = fmaf(bf_hi(u.z), x, acc[5]); acc[6] = fmaf(bf_lo(u.w), x, acc[6]); acc[7] = fmaf(bf_hi(u.w), x, acc[7]);
+    };
+#pragma unroll
+    for (int i = 0; i < LAB_KEEP; ++i)
+      if (grp + 32 * i < p.dim) add(w[i], q[grp + 32 * i]);
+    for (int d = grp + 32 * LAB_KEEP; d < p.dim; d += 32)
+      if (col_ok) add(ldg128(uk + (size_t)d * p.kvp + col), q[d]);
+#pragma unroll
+    for (int e = 0; e < 8; ++e) {
+      acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], 8);
+      acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], 16);
+    }
+    if (lane < 8) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) part[(warp * LAB_BATCH + b) * LAB_COLS + 8 * lane + e] = acc[e];
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < nb * LAB_COLS; i += LAB_THREADS) {
+    const int b = i / LAB_COLS, c = i - b * LAB_COLS, j = blockIdx.x * LAB_COLS + c;
+    if (j >= p.kvp) continue;
+    float t = 0.f;
+#pragma unroll
+    for (int x = 0; x < LAB_THREADS / 32; ++x) t += part[(x * LAB_BATCH + b) * LAB_COLS + c];
+    const size_t at = ((size_t)(b0 + b) * p.heads + h) * a.qrow + j;
+    split_bf16(t, a.q_hi[at], a.q_lo[at]);
+  }
+  if (blockIdx.x) return;
+  // first column block: the rotated part of the queries and, for head 0, the new cache rows
+  for (int b = 0; b < nb; ++b) {
+    const int pos = p.positions[b0 + b];
+    if (pos < 0 || pos >= p.max_ctx) {  // nothing is appended, and the next launch skips the sequence
+      if (h == 0 && tid == 0 && p.error_flag) *reinterpret_cast<volatile int*>(p.error_flag) = 3;
+      continue;
+    }
+    const float* table = p.rope + (size_t)pos * p.pairs * 2;
+    const float* qr = p.q + (size_t)(b0 + b) * p.q_stride + h * qd + p.dim;
+    for (int i = tid; i < a.qrow - p.kvp; i += LAB_THREADS) {
+      const size_t at = ((size_t)(b0 + b) * p.heads + h) * a.qrow + p.kvp + i;
+      split_bf16(i < p.rot_dim ? rotated(qr, i, table, p.pairs) * p.scale : 0.f, a.q_hi[at], a.q_lo[at]);
+    }
+    if (h) continue;
+    const float* in = p.low + (size_t)(b0 + b) * p.low_stride;
+    float ss[1] = {0.f};
+    for (int i = tid; i < p.kv_rank; i += LAB_THREADS) ss[0] += in[i] * in[i];
+    block_sums<1, LAB_THREADS / 32>(ss, red);
+    const float f = 1.0f / sqrtf(ss[0] / (float)p.kv_rank + p.eps);
+    __nv_bfloat16* row = static_cast<__nv_bfloat16*>(p.cache) + ((size_t)p.slots[b0 + b] * p.cap + pos % p.cap) * p.crow;
+    for (int i = tid; i < p.kv_rank; i += LAB_THREADS) row[i] = __float2bfloat16(in[i] * f * p.c_norm[i]);
+    for (int i = tid; i < p.rot_dim; i += LAB_THREADS) row[p.kvp + i] = __float2bfloat16(rotated(in + p.kv_rank, i, table, p.pairs));
+  }
+}
+
+constexpr int LAS_THREADS = 128, LAS_HEADS = 16, LAS_KEYS = 64;
+
+__host__ __device__ __forceinline__ int las_row(int n) { return (n + 15) / 16 * 16; }
+__host__ __device__ __forceinline__ size_t las_smem_bytes(int crow) {
+  const size_t row = las_row(crow) + 8;
+  return (LAS_KEYS + 2 * LAS_HEADS) * row * 2 + (size_t)2 * LAS_HEADS * (LAS_KEYS + 8) * 2;
+}
+
+struct LatentSplitParams {
+  const __nv_bfloat16 *q_hi, *q_lo;  // [batch][heads][qrow]
+  int qrow;
+  const __nv_bfloat16* cache;        // [slot][cap][crow]
+  int crow, kvp, cap;
+  const int* positions;
+  const int* slots;
+  int heads, window, max_ctx, nsplit;
+  float* part_o;                     // [batch][heads][nsplit][kvp]
+  float* part_ml;                    // [batch][heads][nsplit]{max, sum}, base-e scores
+};
+
+// grid = (splits, groups of 16 heads, batch). TW = most 8-column tiles of the weighted sum per warp.
+template <int TW>
+__global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentSplitParams p) {
+  extern __shared__ __align__(16) unsigned char las_smem[];
+  __shared__ float mx_s[4][LAS_HEADS], sum_s[4][LAS_HEADS];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int split = blockIdx.x, h0 = blockIdx.y * LAS_HEADS, b = blockIdx.z;
+  const int EP = las_row(p.crow), RS = EP + 8, PS = LAS_KEYS + 8;
+  __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(las_smem);
+  __nv_bfloat16* Qh = Ks + LAS_KEYS * RS;
+  __nv_bfloat16* Ql = Qh + LAS_HEADS * RS;
+  __nv_bfloat16* Ph = Ql + LAS_HEADS * RS;
+  __nv_bfloat16* Pl = Ph + LAS_HEADS * PS;
+  pdl_launch_dependents();
+  pdl_wait();
+  const int pos = p.positions[b];
+  if (pos < 0 || pos >= p.max_ctx) return;
+  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, nkeys = pos - lo + 1;
+  const int chunk = ((nkeys + p.nsplit - 1) / p.nsplit + LAS_KEYS - 1) / LAS_KEYS * LAS_KEYS;
+  const int k_begin = lo + split * chunk, k_end = min(pos + 1, k_begin + chunk);
+  const __nv_bfloat16* cache = p.cache + (size_t)p.slots[b] * p.cap * p.crow;
+  const int nh = min(LAS_HEADS, p.heads - h0), ce = EP >> 3, cc = p.crow >> 3;
+  for (int i = tid; i < LAS_HEADS * ce; i += LAS_THREADS) {
+    const int r = i / ce, c = i - r * ce;
+    uint4 vh = make_uint4(0, 0, 0, 0), vl = vh;
+    if (r < nh) {
+      const size_t at = ((size_t)b * p.heads + h0 + r) * p.qrow + 8 * c;
+      vh = *reinterpret_cast<const uint4*>(p.q_hi + at);
+      vl = *reinterpret_cast<const uint4*>(p.q_lo + at);
+    }
+    *reinterpret_cast<uint4*>(Qh + r * RS + 8 * c) = vh;
+    *reinterpret_cast<uint4*>(Ql + r * RS + 8 * c) = vl;
+  }
+  const int tiles = p.kvp >> 3;  // 8-column tiles of the weighted sum; a warp takes pairs of them
+  float o[TW][4];
+#pragma unroll
+  for (int i = 0; i < TW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // heads g and g + 8
+  for (int kt = k_begin; kt < k_end; kt += LAS_KEYS) {
+    const int nk = min(LAS_KEYS, k_end - kt);
+    __syncthreads();
+    for (int i = tid; i < LAS_KEYS * ce; i += LAS_THREADS) {
+      const int r = i / ce, c = i - r * ce;
+      __nv_bfloat16* d = Ks + r * RS + 8 * c;
+      if (r < nk && c < cc) pfa_cp16(d, cache + (size_t)((kt + r) % p.cap) * p.crow + 8 * c);
+      else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+    }
+    pfa_cp_wait_all();
+    __syncthreads();
+    // scores of this warp's 16 keys
+    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
+#pragma unroll 4
+    for (int ks = 0; ks < EP; ks += 16) {
+      uint32_t ah[4], al[4], kb[4];
+      const int aoff = (lane & 15) * RS + ks + (lane >> 4) * 8;
+      pfa_ldm4(ah, Qh + aoff);
+      pfa_ldm4(al, Ql + aoff);
+      pfa_ldm4(kb, Ks + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * RS + ks + ((lane >> 3) & 1) * 8);
+      lap_mma(s[0], ah, kb[0], kb[1]);
+      lap_mma(s[1], ah, kb[2], kb[3]);
+      lap_mma(s[0], al, kb[0], kb[1]);
+      lap_mma(s[1], al, kb[2], kb[3]);
+    }
+    float x0 = -INFINITY, x1 = -INFINITY;
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        if (warp * 16 + 8 * i + 2 * t + e >= nk) s[i][e] = s[i][2 + e] = -INFINITY;
+        x0 = fmaxf(x0, s[i][e]);
+        x1 = fmaxf(x1, s[i][2 + e]);
+      }
+#pragma unroll
+    for (int x = 1; x < 4; x <<= 1) {
+      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, x));
+      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, x));
+    }
+    if (t == 0) { mx_s[warp][g] = x0; mx_s[warp][g + 8] = x1; }
+    __syncthreads();
+    const float n0 = fmaxf(m0, fmaxf(fmaxf(mx_s[0][g], mx_s[1][g]), fmaxf(mx_s[2][g], mx_s[3][g])));
+    const float n1 = fmaxf(m1, fmaxf(fmaxf(mx_s[0][g + 8], mx_s[1][g + 8]), fmaxf(mx_s[2][g + 8], mx_s[3][g + 8])));
+    const float f0 = expf(m0 - n0), f1 = expf(m1 - n1);  // every tile has a key, so n is finite
+    m0 = n0; m1 = n1;
+    float y0 = 0.f, y1 = 0.f;
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int k = warp * 16 + 8 * i + 2 * t + e;
+        const float w0 = expf(s[i][e] - n0), w1 = expf(s[i][2 + e] - n1);
+        y0 += w0; y1 += w1;
+        split_bf16(w0, Ph[g * PS + k], Pl[g * PS + k]);
+        split_bf16(w1, Ph[(g + 8) * PS + k], Pl[(g + 8) * PS + k]);
+      }
+    l0 = l0 * f0 + y0; l1 = l1 * f1 + y1;  // this thread's share; shares of lanes and warps are added at the end
+#pragma unroll
+    for (int i = 0; i < TW; ++i) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
+    __syncthreads();
+    // weighted sums: this warp's pairs of column tiles
+#pragma unroll
+    for (int kk = 0; kk < 4; ++kk) {
+      uint32_t ah[4], al[4];
+      const int aoff = (lane & 15) * PS + kk * 16 + (lane >> 4) * 8;
+      pfa_ldm4(ah, Ph + aoff);
+      pfa_ldm4(al, Pl + aoff);
+#pragma unroll
+      for (int i = 0; i < TW / 2; ++i) {
+        const int tile = 2 * (warp + 4 * i);
+        if (tile < tiles) {  // an odd last tile reads the row's next eight columns and drops them
+          uint32_t vb[4];
+          pfa_ldm4t(vb, Ks + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RS + tile * 8 + (lane >> 4) * 8);
+          lap_mma(o[2 * i], ah, vb[0], vb[1]);
+          lap_mma(o[2 * i + 1], ah, vb[2], vb[3]);
+          lap_mma(o[2 * i], al, vb[0], vb[1]);
+          lap_mma(o[2 * i + 1], al, vb[2], vb[3]);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int x = 1; x < 4; x <<= 1) {
+    l0 += __shfl_xor_sync(0xffffffffu, l0, x);
+    l1 += __shfl_xor_sync(0xffffffffu, l1, x);
+  }
+  __syncthreads();
+  if (t == 0) { sum_s[warp][g] = l0; sum_s[warp][g + 8] = l1; mx_s[warp][g] = m0; mx_s[warp][g + 8] = m1; }
+  __syncthreads();
+  const size_t row = ((size_t)b * p.heads + h0) * p.nsplit + split;
+  if (tid < nh) {
+    float* ml = p.part_ml + (row + (size_t)tid * p.nsplit) * 2;
+    ml[0] = mx_s[0][tid];
+    ml[1] = k_begin < k_end ? sum_s[0][tid] + sum_s[1][tid] + sum_s[2][tid] + sum_s[3][tid] : 0.f;
+  }
+  if (k_begin >= k_end) return;  // an empty run: its sum of zero makes the merge skip it
+#pragma unroll
+  for (int i = 0; i < TW; ++i) {
+    const int tile = 2 * (warp + 4 * (i >> 1)) + (i & 1);
+    if (tile < tiles) {
+      const int c = 8 * tile + 2 * t;
+      if (g < nh) *reinterpret_cast<float2*>(p.part_o + (row + (size_t)g * p.nsplit) * p.kvp + c) = make_float2(o[i][0], o[i][1]);
+      if (g + 8 < nh) *reinterpret_cast<float2*>(p.part_o + (row + (size_t)(g + 8) * p.nsplit) * p.kvp + c) = make_float2(o[i][2], o[i][3]);
+    }
+  }
+}
+
+constexpr int LAM_THREADS = 256, LAM_ROWS = 32;  // value rows per block: four per warp
+constexpr int LAM_KEEP = 4;                      // pieces of each W_uv row a lane requests ahead (kv_rank up to 1024)
+
+// grid = (vdim / 32 rounded up, heads, batch). O = type of the output rows.
+template <typename O>
+__global__ void __launch_bounds__(LAM_THREADS) latent_merge_kernel(const LatentDecodeParams p) {
+  extern __shared__ __align__(16) float lam_s[];  // merged sum of latents [kvp], normalised
+  __shared__ float w_s[LAD_MAX_SPLITS];
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, b = blockIdx.z;
+  const int r0 = blockIdx.x * LAM_ROWS + warp * 4, vch = p.kvp >> 3;
+  pdl_launch_dependents();
+  const __nv_bfloat16* uv = p.uv + (size_t)h * p.vdim * p.kvp;
+  uint4 w[4][LAM_KEEP];
+#pragma unroll
+  for (int e = 0; e < 4; ++e)
+#pragma unroll
+    for (int i = 0; i < LAM_KEEP; ++i)
+      w[e][i] = lane + 32 * i < vch && r0 + e < p.vdim ? ldg128(uv + (size_t)(r0 + e) * p.kvp + 8 * (lane + 32 * i)) : make_uint4(0, 0, 0, 0);
+  pdl_wait();
+  const int pos = p.positions[b];
+  if (pos < 0 || pos >= p.max_ctx) return;
+  const size_t base = ((size_t)b * p.heads + h) * p.nsplit;
+  if (warp == 0) {  // weight of every run: exp(its max - the largest max) / total sum
+    float m[LAD_MAX_SPLITS / 32], l[LAD_MAX_SPLITS / 32], M = -INFINITY, L = 0.f;
+#pragma unroll
+    for (int i = 0; i < LAD_MAX_SPLITS / 32; ++i) {
+      const int s = lane + 32 * i;
+      const float2 ml = s < p.nsplit ? __ldcg(reinterpret_cast<const float2*>(p.part_ml + (base + s) * 2)) : make_float2(0.f, 0.f);
+      m[i] = ml.x; l[i] = ml.y;
+      if (l[i] > 0.f) M = fmaxf(M, m[i]);
+    }
+    M = warp_max(M);
+#pragma unroll
+    for (int i = 0; i < LAD_MAX_SPLITS / 32; ++i) {
+      m[i] = l[i] > 0.f ? expf(m[i] - M) : 0.f;
+      L += m[i] * l[i];
+    }
+    L = warp_sum(L);
+#pragma unroll
+    for (int i = 0; i < LAD_MAX_SPLITS / 32; ++i) w_s[lane + 32 * i] = m[i] / L;
+  }
+  __syncthreads();
+  for (int i = tid; i < p.kvp; i += LAM_THREADS) {
+    float o = 0.f;
+#pragma unroll 8
+    for (int s = 0; s < p.nsplit; ++s)
+      if (w_s[s] > 0.f) o = fmaf(w_s[s], __ldcg(p.part_o + (base + s) * p.kvp + i), o);
+    lam_s[i] = o;
+  }
+  __syncthreads();
+  float acc[4] = {0.f, 0.f, 0.f, 0.f};
+  auto add = [&](int e, const uint4& u, const float* x) {
+    acc[e] = fmaf(bf_lo(u.x), x[0], acc[e]); acc[e] = fmaf(bf_hi(u.x), x[1], acc[e]); acc[e] = fmaf(bf_lo(u.y), x[2], acc[e]); acc[e] = fmaf(bf_hi(u.y), x[3], acc[e]);
+    acc[e] = fmaf(bf_lo(u.z), x[4], acc[e]); acc[e] = fmaf(bf_hi(u.z), x[5], acc[e]); acc[e] = fmaf(bf_lo(u.w), x[6], acc[e]); acc[e] = fmaf(bf_hi(u.w), x[7], acc[e]);
+  };
+#pragma unroll
+  for (int i = 0; i < LAM_KEEP; ++i)
+    if (lane + 32 * i < vch) {
+      float x[8];
+      load8(lam_s + 8 * (lane + 32 * i), x);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) add(e, w[e][i], x);
+    }
+  for (int c = lane + 32 * LAM_KEEP; c < vch; c += 32) {
+    float x[8];
+    load8(lam_s + 8 * c, x);
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (r0 + e < p.vdim) add(e, ldg128(uv + (size_t)(r0 + e) * p.kvp + 8 * c), x);
+  }
+#pragma unroll
+  for (int e = 0; e < 4; ++e) acc[e] = warp_sum(acc[e]);
+  if (lane < 4 && r0 + lane < p.vdim) {
+    const float v = lane == 0 ? acc[0] : lane == 1 ? acc[1] : lane == 2 ? acc[2] : acc[3];
+    const int j = h * p.vdim + r0 + lane;
+    static_cast<O*>(p.out)[(size_t)b * p.out_stride + j] = to_operand<O>(v * p.gate[(size_t)b * p.gate_stride + j]);
+  }
+}
+
 // ---- prompts -----------------------------------------------------------------------------------------------------
 constexpr int LAP_Q = 64, LAP_K = 64, LAP_THREADS = 128;
 
@@ -363,17 +727,6 @@ struct LatentPrefillParams {
 __host__ __device__ __forceinline__ int lap_qk_stride(int dim, int rot) { return (dim + rot + 15) / 16 * 16 + 8; }
 __host__ __device__ __forceinline__ size_t lap_smem_bytes(int dim, int rot, int vp) {
   return ((size_t)(LAP_Q + LAP_K) * lap_qk_stride(dim, rot) + (size_t)LAP_K * (vp + 8)) * 2;
-}
-
-__device__ __forceinline__ void lap_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<const uint32_t*>(&v);
 }
 
 // grid = (query blocks of the longest run, heads, runs). VP = value columns per head rounded up to 32, 64, 128 or 256.

@@ -9,6 +9,8 @@
 //
 // State of a slot: [head][key][value]. A token at position 0 starts from zeros whatever the slot held before.
 #pragma once
+#include <type_traits>
+
 #include "block_rows.cuh"
 
 namespace b200 {
@@ -99,6 +101,7 @@ __global__ void __launch_bounds__(WKV_STEP_THREADS) wkv_step_kernel(const WkvSte
 constexpr int WKV_SCAN_THREADS = 128;
 constexpr int WKV_TILE = 16;  // tokens staged per step
 constexpr int WKV_KPT = 8;    // keys per thread
+constexpr int WKV_NC = 2;     // value columns per thread
 
 struct WkvScanParams {
   const float* rkv;    // [T][stride]: r, k, v at offsets 0, off, 2 off
@@ -124,89 +127,131 @@ __host__ __device__ __forceinline__ int wkv_lanes(int dim) {
   while (l * WKV_KPT < dim) l *= 2;
   return l;
 }
-__host__ __device__ __forceinline__ int wkv_cols(int dim) { return WKV_SCAN_THREADS / wkv_lanes(dim); }
+__host__ __device__ __forceinline__ int wkv_cols(int dim) { return WKV_NC * WKV_SCAN_THREADS / wkv_lanes(dim); }
 __host__ __device__ __forceinline__ size_t wkv_scan_smem(int dim) {
   return (size_t)2 * WKV_TILE * (3 * wkv_lanes(dim) * WKV_KPT + wkv_cols(dim)) * 4;
 }
 
-// grid = (column blocks of a head, heads, runs). L = lanes per column.
+// grid = (column blocks of a head, heads, runs). L = lanes per column; a thread has two columns, COLS / 2 apart.
 template <int L>
 __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvScanParams p) {
-  extern __shared__ __align__(16) float scan_s[];  // two tiles of [token][r | k | w (DP each) | v (cols)]
-  constexpr int DP = L * WKV_KPT, COLS = WKV_SCAN_THREADS / L, ROW = 3 * DP + COLS;
-  const int tid = threadIdx.x, h = blockIdx.y, D = p.dim, hc = h * D;
+  extern __shared__ __align__(16) float scan_s[];  // two tiles of [token][r | k | w (DP each) | v (COLS)]
+  constexpr int DP = L * WKV_KPT, HALF = WKV_SCAN_THREADS / L, COLS = WKV_NC * HALF, ROW = 3 * DP + COLS;
+  constexpr int G = L < WKV_TILE ? L : WKV_TILE;   // tokens whose outputs are reduced together
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, D = p.dim, hc = h * D;
   const RunDesc run = p.runs[blockIdx.z];
-  const int ln = tid % L, col = blockIdx.x * COLS + tid / L;
-  const bool col_ok = col < D;
+  const int ln = tid % L, cl = tid / L, c0 = blockIdx.x * COLS;  // columns c0 + cl and c0 + cl + HALF
   const int k0 = ln * WKV_KPT;
   float* S = p.state + ((size_t)run.slot * p.heads + h) * D * D;
-  float st[WKV_KPT], u[WKV_KPT];
+  float st[WKV_NC][WKV_KPT], u[WKV_KPT];
 #pragma unroll
   for (int i = 0; i < WKV_KPT; ++i) {
     const int k = k0 + i;
     u[i] = k < D ? p.u[hc + k] : 0.f;
-    st[i] = run.start > 0 && k < D && col_ok ? S[(size_t)k * D + col] : 0.f;
+#pragma unroll
+    for (int n = 0; n < WKV_NC; ++n) {
+      const int col = c0 + cl + n * HALF;
+      st[n][i] = run.start > 0 && k < D && col < D ? S[(size_t)k * D + col] : 0.f;
+    }
   }
   // padding keys and columns stay zero in both tiles
   for (int i = tid; i < 2 * WKV_TILE * ROW; i += WKV_SCAN_THREADS) scan_s[i] = 0.f;
   __syncthreads();
   const bool vec = !((D | hc | p.stride | p.off | p.decay_stride) & 3);  // 16-byte pieces possible
-  auto fetch = [&](int tile) {
-    float* dst = scan_s + (size_t)(tile & 1) * WKV_TILE * ROW;
+  const int nv = min(COLS, D - c0);
+  auto cp4 = [](float* dst, const float* src) {
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((uint32_t)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+  };
+  auto fetch = [&](int tile) {  // a warp takes every fourth token of the tile
     const int first = tile * WKV_TILE, n = min(WKV_TILE, run.len - first);
-    if (n <= 0) return;
-    const int per = vec ? D / 4 : D;
-    for (int i = tid; i < n * 3 * per; i += WKV_SCAN_THREADS) {
-      const int t = i / (3 * per), e = i - t * 3 * per, which = e / per, c = e - which * per;
+    for (int t = warp; t < n; t += WKV_SCAN_THREADS / 32) {
+      float* d = scan_s + (size_t)((tile & 1) * WKV_TILE + t) * ROW;
       const size_t row = (size_t)(run.row0 + first + t);
-      const float* src = which == 2 ? p.decay + row * p.decay_stride + hc : p.rkv + row * p.stride + which * p.off + hc;
-      float* d = dst + t * ROW + which * DP;
-      if (vec) pfa_cp16(d + 4 * c, src + 4 * c);
-      else d[c] = src[c];
+      const float* rk = p.rkv + row * p.stride + hc;
+      const float* dec = p.decay + row * p.decay_stride + hc;
+      if (vec) {
+        for (int c = lane * 4; c < D; c += 128) {
+          pfa_cp16(d + c, rk + c);
+          pfa_cp16(d + DP + c, rk + p.off + c);
+          pfa_cp16(d + 2 * DP + c, dec + c);
+        }
+      } else {
+        for (int c = lane; c < D; c += 32) {
+          cp4(d + c, rk + c);
+          cp4(d + DP + c, rk + p.off + c);
+          cp4(d + 2 * DP + c, dec + c);
+        }
+      }
+      for (int c = lane; c < nv; c += 32) cp4(d + 3 * DP + c, rk + 2 * p.off + c0 + c);
     }
-    for (int i = tid; i < n * COLS; i += WKV_SCAN_THREADS) {
-      const int t = i / COLS, c = i - t * COLS;
-      if (blockIdx.x * COLS + c < D) dst[t * ROW + 3 * DP + c] = p.rkv[(size_t)(run.row0 + first + t) * p.stride + 2 * p.off + hc + blockIdx.x * COLS + c];
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
   };
   const int tiles = (run.len + WKV_TILE - 1) / WKV_TILE;
   fetch(0);
   for (int tile = 0; tile < tiles; ++tile) {
     pfa_cp_wait_all();
     __syncthreads();  // the tile has landed for everyone, and everyone has left the other buffer
-    fetch(tile + 1);
+    if (tile + 1 < tiles) fetch(tile + 1);
     const float* base = scan_s + (size_t)(tile & 1) * WKV_TILE * ROW;
     const int n = min(WKV_TILE, run.len - tile * WKV_TILE);
-    float mine = 0.f;  // outputs are written L tokens at a time, one per lane of the column
-#pragma unroll 4
-    for (int t = 0; t < n; ++t) {
-      const float* row = base + t * ROW;
-      const float4 r0 = *reinterpret_cast<const float4*>(row + k0), r1 = *reinterpret_cast<const float4*>(row + k0 + 4);
-      const float4 a0 = *reinterpret_cast<const float4*>(row + DP + k0), a1 = *reinterpret_cast<const float4*>(row + DP + k0 + 4);
-      const float4 w0 = *reinterpret_cast<const float4*>(row + 2 * DP + k0), w1 = *reinterpret_cast<const float4*>(row + 2 * DP + k0 + 4);
-      const float v = row[3 * DP + tid / L];
-      const float r[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
-      const float k[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
-      const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
-      float o = 0.f;
+    auto group = [&](int g0, auto whole) {  // tokens g0 .. g0 + G - 1 of the tile
+      float o[WKV_NC][G];
 #pragma unroll
-      for (int i = 0; i < WKV_KPT; ++i) {
-        const float kv = k[i] * v;
-        o = fmaf(r[i], fmaf(u[i], kv, st[i]), o);
-        st[i] = fmaf(w[i], st[i], kv);
+      for (int j = 0; j < G; ++j) {
+#pragma unroll
+        for (int c = 0; c < WKV_NC; ++c) o[c][j] = 0.f;
+        if (!decltype(whole)::value && g0 + j >= n) continue;
+        const float* row = base + (g0 + j) * ROW;
+        const float4 r0 = *reinterpret_cast<const float4*>(row + k0), r1 = *reinterpret_cast<const float4*>(row + k0 + 4);
+        const float4 a0 = *reinterpret_cast<const float4*>(row + DP + k0), a1 = *reinterpret_cast<const float4*>(row + DP + k0 + 4);
+        const float4 w0 = *reinterpret_cast<const float4*>(row + 2 * DP + k0), w1 = *reinterpret_cast<const float4*>(row + 2 * DP + k0 + 4);
+        const float r[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
+        const float k[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
+        const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+#pragma unroll
+        for (int c = 0; c < WKV_NC; ++c) {
+          const float v = row[3 * DP + cl + c * HALF];
+          float x = 0.f, y = 0.f;  // two chains
+#pragma unroll
+          for (int i = 0; i < WKV_KPT; ++i) {
+            const float kv = k[i] * v;
+            float& acc = i & 1 ? y : x;
+            acc = fmaf(r[i], fmaf(u[i], kv, st[c][i]), acc);
+            st[c][i] = fmaf(w[i], st[c][i], kv);
+          }
+          o[c][j] = x + y;
+        }
       }
+      // sums over the column's lanes; lane j (mod G) ends up with token j
 #pragma unroll
-      for (int s = L / 2; s > 0; s >>= 1) o += __shfl_xor_sync(0xffffffffu, o, s);
-      if (t % L == ln) mine = o;
-      if ((t % L == L - 1 || t == n - 1) && col_ok && ln <= t % L)
-        p.o[(size_t)(run.row0 + tile * WKV_TILE + t - t % L + ln) * p.o_stride + hc + col] = mine;
-    }
+      for (int c = 0; c < WKV_NC; ++c) {
+        if (L > G)
+#pragma unroll
+          for (int j = 0; j < G; ++j) o[c][j] += __shfl_xor_sync(0xffffffffu, o[c][j], L / 2);
+#pragma unroll
+        for (int s = G / 2; s > 0; s >>= 1)
+#pragma unroll
+          for (int j = 0; j < s; ++j) {
+            const bool up = ln & s;
+            const float send = up ? o[c][j] : o[c][j + s], keep = up ? o[c][j + s] : o[c][j];
+            o[c][j] = keep + __shfl_xor_sync(0xffffffffu, send, s);
+          }
+        const int t = g0 + ln % G, col = c0 + cl + c * HALF;
+        if (ln < G && t < n && col < D) p.o[(size_t)(run.row0 + tile * WKV_TILE + t) * p.o_stride + hc + col] = o[c][0];
+      }
+    };
+    if (n == WKV_TILE)
+      for (int g0 = 0; g0 < WKV_TILE; g0 += G) group(g0, std::true_type{});
+    else
+      for (int g0 = 0; g0 < n; g0 += G) group(g0, std::false_type{});
   }
-  if (col_ok)
 #pragma unroll
-    for (int i = 0; i < WKV_KPT; ++i)
-      if (k0 + i < D) S[(size_t)(k0 + i) * D + col] = st[i];
+  for (int n = 0; n < WKV_NC; ++n) {
+    const int col = c0 + cl + n * HALF;
+    if (col < D)
+#pragma unroll
+      for (int i = 0; i < WKV_KPT; ++i)
+        if (k0 + i < D) S[(size_t)(k0 + i) * D + col] = st[n][i];
+  }
   if (blockIdx.x == 0) {  // the heads' first blocks share the copy of the last token's h
     const float* src = p.h + (size_t)(run.row0 + run.len - 1) * p.h_stride;
     float* dst = p.shift + ((size_t)run.slot * 2 + ((run.start + run.len) & 1)) * p.shift_stride;
