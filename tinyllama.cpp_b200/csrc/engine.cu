@@ -699,11 +699,10 @@ static int packed_forward_step(b200_engine* e, int batch, int nsplit, cudaStream
 // The launch sequence of one decode step for `batch` sequences (also what gets captured): the model's layers and
 // logits, then token selection. Returns the number of kernel launches.
 static int enqueue_step(b200_engine* e, int batch, int nsplit, cudaStream_t st, bool with_embed, int* head_ctas_out, bool penalized = false) {
-  const bool rows = batch >= e->gemm_min_batch;
+  const bool rows = batch >= (e->blocks && penalized ? PEN_MAX_BATCH + 1 : e->gemm_min_batch);
   const bool peer = e->tp_size > 1 && e->use_peer && !rows;
   int parts = 0, launches;
   if (e->blocks) {
-    if (rows && penalized) throw std::runtime_error("the repetition penalty of the device loop is built for the matvec path (batch < " + std::to_string(e->gemm_min_batch) + ")");
     launches = rows ? block_forward_batch(e, batch, st, with_embed, &parts) : block_forward_step(e, batch, st, with_embed, penalized, &parts);
   } else {
     launches = packed_forward_step(e, batch, nsplit, st, with_embed, penalized, &parts);

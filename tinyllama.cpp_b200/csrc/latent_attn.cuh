@@ -5,7 +5,7 @@
 //
 //   latent_append_kernel   prompts: norm + rotation of new rows into the ring, and the rows a chunk attends to laid out
 //                          contiguously (history from the ring, then the new ones) for the key / value expansion
-//   latent_prefill_kernel  prompts: 64 queries of one head per block over expanded keys and values, 64-key tiles, online
+//   latent_prefill_kernel  prompts: 128 queries of one head per block over expanded keys and values, 64-key tiles, online
 //                          softmax, bfloat16 tensor-core products (mma.sync m16n8k16) with FP32 scores and sums
 //   decode                 one token of several sequences: works on the latents themselves. The query's unrotated part is
 //                          taken through W_uk once (q . W_uk c = (W_uk^T q) . c), scores and the weighted sum run over c,
@@ -375,7 +375,8 @@ struct LatentAbsorbParams {
   int qrow, batch;
 };
 
-// grid = (kvp / 64 rounded up, heads, batch / 8 rounded up)
+// grid = (kvp / 64 rounded up, then one more, heads, batch / 8 rounded up): the last block of a head rotates the queries'
+// other part and, for head 0, appends the new cache rows while the others go through W_uk.
 __global__ void __launch_bounds__(LAB_THREADS) latent_absorb_kernel(const LatentAbsorbParams a) {
   const LatentDecodeParams& p = a.d;
   extern __shared__ __align__(16) float lab_s[];  // queries [LAB_BATCH][dim], then partial sums [8 warps][LAB_BATCH][64]
@@ -384,6 +385,33 @@ __global__ void __launch_bounds__(LAB_THREADS) latent_absorb_kernel(const Latent
   const int b0 = blockIdx.z * LAB_BATCH, nb = min(LAB_BATCH, a.batch - b0);
   float* part = lab_s + LAB_BATCH * p.dim;
   pdl_launch_dependents();
+  const int qd = p.dim + p.rot_dim;
+  if (blockIdx.x * LAB_COLS >= p.kvp) {
+    pdl_wait();
+    for (int b = 0; b < nb; ++b) {
+      const int pos = p.positions[b0 + b];
+      if (pos < 0 || pos >= p.max_ctx) {  // nothing is appended, and the next launch skips the sequence
+        if (h == 0 && tid == 0 && p.error_flag) *reinterpret_cast<volatile int*>(p.error_flag) = 3;
+        continue;
+      }
+      const float* table = p.rope + (size_t)pos * p.pairs * 2;
+      const float* qr = p.q + (size_t)(b0 + b) * p.q_stride + h * qd + p.dim;
+      for (int i = tid; i < a.qrow - p.kvp; i += LAB_THREADS) {
+        const size_t at = ((size_t)(b0 + b) * p.heads + h) * a.qrow + p.kvp + i;
+        split_bf16(i < p.rot_dim ? rotated(qr, i, table, p.pairs) * p.scale : 0.f, a.q_hi[at], a.q_lo[at]);
+      }
+      if (h) continue;
+      const float* in = p.low + (size_t)(b0 + b) * p.low_stride;
+      float ss[1] = {0.f};
+      for (int i = tid; i < p.kv_rank; i += LAB_THREADS) ss[0] += in[i] * in[i];
+      block_sums<1, LAB_THREADS / 32>(ss, red);
+      const float f = 1.0f / sqrtf(ss[0] / (float)p.kv_rank + p.eps);
+      __nv_bfloat16* row = static_cast<__nv_bfloat16*>(p.cache) + ((size_t)p.slots[b0 + b] * p.cap + pos % p.cap) * p.crow;
+      for (int i = tid; i < p.kv_rank; i += LAB_THREADS) row[i] = __float2bfloat16(in[i] * f * p.c_norm[i]);
+      for (int i = tid; i < p.rot_dim; i += LAB_THREADS) row[p.kvp + i] = __float2bfloat16(rotated(in + p.kv_rank, i, table, p.pairs));
+    }
+    return;
+  }
   // thread = (8 columns, every 32nd row of the head's W_uk): pieces requested before anything else
   const int ch = tid & 7, grp = tid >> 3, col = blockIdx.x * LAB_COLS + 8 * ch;
   const bool col_ok = col < p.kvp;
@@ -395,7 +423,6 @@ __global__ void __launch_bounds__(LAB_THREADS) latent_absorb_kernel(const Latent
     w[i] = col_ok && d < p.dim ? ldg128(uk + (size_t)d * p.kvp + col) : make_uint4(0, 0, 0, 0);
   }
   pdl_wait();
-  const int qd = p.dim + p.rot_dim;
   for (int i = tid; i < nb * p.dim; i += LAB_THREADS) {
     const int b = i / p.dim, d = i - b * p.dim;
     lab_s[i] = p.q[(size_t)(b0 + b) * p.q_stride + h * qd + d] * p.scale;
@@ -433,35 +460,11 @@ __global__ void __launch_bounds__(LAB_THREADS) latent_absorb_kernel(const Latent
     const size_t at = ((size_t)(b0 + b) * p.heads + h) * a.qrow + j;
     split_bf16(t, a.q_hi[at], a.q_lo[at]);
   }
-  if (blockIdx.x) return;
-  // first column block: the rotated part of the queries and, for head 0, the new cache rows
-  for (int b = 0; b < nb; ++b) {
-    const int pos = p.positions[b0 + b];
-    if (pos < 0 || pos >= p.max_ctx) {  // nothing is appended, and the next launch skips the sequence
-      if (h == 0 && tid == 0 && p.error_flag) *reinterpret_cast<volatile int*>(p.error_flag) = 3;
-      continue;
-    }
-    const float* table = p.rope + (size_t)pos * p.pairs * 2;
-    const float* qr = p.q + (size_t)(b0 + b) * p.q_stride + h * qd + p.dim;
-    for (int i = tid; i < a.qrow - p.kvp; i += LAB_THREADS) {
-      const size_t at = ((size_t)(b0 + b) * p.heads + h) * a.qrow + p.kvp + i;
-      split_bf16(i < p.rot_dim ? rotated(qr, i, table, p.pairs) * p.scale : 0.f, a.q_hi[at], a.q_lo[at]);
-    }
-    if (h) continue;
-    const float* in = p.low + (size_t)(b0 + b) * p.low_stride;
-    float ss[1] = {0.f};
-    for (int i = tid; i < p.kv_rank; i += LAB_THREADS) ss[0] += in[i] * in[i];
-    block_sums<1, LAB_THREADS / 32>(ss, red);
-    const float f = 1.0f / sqrtf(ss[0] / (float)p.kv_rank + p.eps);
-    __nv_bfloat16* row = static_cast<__nv_bfloat16*>(p.cache) + ((size_t)p.slots[b0 + b] * p.cap + pos % p.cap) * p.crow;
-    for (int i = tid; i < p.kv_rank; i += LAB_THREADS) row[i] = __float2bfloat16(in[i] * f * p.c_norm[i]);
-    for (int i = tid; i < p.rot_dim; i += LAB_THREADS) row[p.kvp + i] = __float2bfloat16(rotated(in + p.kv_rank, i, table, p.pairs));
-  }
 }
 
-constexpr int LAS_THREADS = 128, LAS_HEADS = 16, LAS_KEYS = 64;
+constexpr int LAS_THREADS = 256, LAS_WARPS = 8, LAS_HEADS = 16, LAS_KEYS = 64;
 
-__host__ __device__ __forceinline__ int las_row(int n) { return (n + 15) / 16 * 16; }
+__host__ __device__ __forceinline__ int las_row(int n) { return (n + 31) / 32 * 32; }
 __host__ __device__ __forceinline__ size_t las_smem_bytes(int crow) {
   const size_t row = las_row(crow) + 8;
   return (LAS_KEYS + 2 * LAS_HEADS) * row * 2 + (size_t)2 * LAS_HEADS * (LAS_KEYS + 8) * 2;
@@ -483,7 +486,7 @@ struct LatentSplitParams {
 template <int TW>
 __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentSplitParams p) {
   extern __shared__ __align__(16) unsigned char las_smem[];
-  __shared__ float mx_s[4][LAS_HEADS], sum_s[4][LAS_HEADS];
+  __shared__ float mx_s[LAS_WARPS][LAS_HEADS], sum_s[LAS_WARPS][LAS_HEADS];
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int split = blockIdx.x, h0 = blockIdx.y * LAS_HEADS, b = blockIdx.z;
   const int EP = las_row(p.crow), RS = EP + 8, PS = LAS_KEYS + 8;
@@ -501,16 +504,17 @@ __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentS
   const int k_begin = lo + split * chunk, k_end = min(pos + 1, k_begin + chunk);
   const __nv_bfloat16* cache = p.cache + (size_t)p.slots[b] * p.cap * p.crow;
   const int nh = min(LAS_HEADS, p.heads - h0), ce = EP >> 3, cc = p.crow >> 3;
-  for (int i = tid; i < LAS_HEADS * ce; i += LAS_THREADS) {
-    const int r = i / ce, c = i - r * ce;
-    uint4 vh = make_uint4(0, 0, 0, 0), vl = vh;
-    if (r < nh) {
-      const size_t at = ((size_t)b * p.heads + h0 + r) * p.qrow + 8 * c;
-      vh = *reinterpret_cast<const uint4*>(p.q_hi + at);
-      vl = *reinterpret_cast<const uint4*>(p.q_lo + at);
+  for (int r = warp; r < LAS_HEADS; r += LAS_WARPS) {
+    const size_t at = ((size_t)b * p.heads + h0 + min(r, nh - 1)) * p.qrow;
+    for (int c = lane; c < ce; c += 32) {
+      if (r < nh) {
+        pfa_cp16(Qh + r * RS + 8 * c, p.q_hi + at + 8 * c);
+        pfa_cp16(Ql + r * RS + 8 * c, p.q_lo + at + 8 * c);
+      } else {
+        *reinterpret_cast<uint4*>(Qh + r * RS + 8 * c) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(Ql + r * RS + 8 * c) = make_uint4(0, 0, 0, 0);
+      }
     }
-    *reinterpret_cast<uint4*>(Qh + r * RS + 8 * c) = vh;
-    *reinterpret_cast<uint4*>(Ql + r * RS + 8 * c) = vl;
   }
   const int tiles = p.kvp >> 3;  // 8-column tiles of the weighted sum; a warp takes pairs of them
   float o[TW][4];
@@ -520,37 +524,41 @@ __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentS
   for (int kt = k_begin; kt < k_end; kt += LAS_KEYS) {
     const int nk = min(LAS_KEYS, k_end - kt);
     __syncthreads();
-    for (int i = tid; i < LAS_KEYS * ce; i += LAS_THREADS) {
-      const int r = i / ce, c = i - r * ce;
-      __nv_bfloat16* d = Ks + r * RS + 8 * c;
-      if (r < nk && c < cc) pfa_cp16(d, cache + (size_t)((kt + r) % p.cap) * p.crow + 8 * c);
-      else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+    for (int r = warp; r < LAS_KEYS; r += LAS_WARPS) {
+      const __nv_bfloat16* src = cache + (size_t)((kt + r) % p.cap) * p.crow;
+      __nv_bfloat16* d = Ks + r * RS;
+      for (int c = lane; c < ce; c += 32) {
+        if (r < nk && c < cc) pfa_cp16(d + 8 * c, src + 8 * c);
+        else *reinterpret_cast<uint4*>(d + 8 * c) = make_uint4(0, 0, 0, 0);
+      }
     }
     pfa_cp_wait_all();
     __syncthreads();
-    // scores of this warp's 16 keys
-    float s[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-#pragma unroll 4
-    for (int ks = 0; ks < EP; ks += 16) {
-      uint32_t ah[4], al[4], kb[4];
+    // scores of this warp's 8 keys
+    float s[4] = {0.f, 0.f, 0.f, 0.f}, sl[4] = {0.f, 0.f, 0.f, 0.f};  // products with the queries' values and remainders
+#pragma unroll 2
+    for (int ks = 0; ks < EP; ks += 32) {
+      uint32_t a0[4], a1[4], b0[4], b1[4], kb[4];
       const int aoff = (lane & 15) * RS + ks + (lane >> 4) * 8;
-      pfa_ldm4(ah, Qh + aoff);
-      pfa_ldm4(al, Ql + aoff);
-      pfa_ldm4(kb, Ks + (warp * 16 + (lane & 7) + (lane >> 4) * 8) * RS + ks + ((lane >> 3) & 1) * 8);
-      lap_mma(s[0], ah, kb[0], kb[1]);
-      lap_mma(s[1], ah, kb[2], kb[3]);
-      lap_mma(s[0], al, kb[0], kb[1]);
-      lap_mma(s[1], al, kb[2], kb[3]);
+      pfa_ldm4(kb, Ks + (warp * 8 + (lane & 7)) * RS + ks + (lane >> 3) * 8);
+      pfa_ldm4(a0, Qh + aoff);
+      pfa_ldm4(a1, Qh + aoff + 16);
+      pfa_ldm4(b0, Ql + aoff);
+      pfa_ldm4(b1, Ql + aoff + 16);
+      lap_mma(s, a0, kb[0], kb[1]);
+      lap_mma(sl, b0, kb[0], kb[1]);
+      lap_mma(s, a1, kb[2], kb[3]);
+      lap_mma(sl, b1, kb[2], kb[3]);
     }
     float x0 = -INFINITY, x1 = -INFINITY;
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        if (warp * 16 + 8 * i + 2 * t + e >= nk) s[i][e] = s[i][2 + e] = -INFINITY;
-        x0 = fmaxf(x0, s[i][e]);
-        x1 = fmaxf(x1, s[i][2 + e]);
-      }
+    for (int e = 0; e < 2; ++e) {
+      const bool ok = warp * 8 + 2 * t + e < nk;
+      s[e] = ok ? s[e] + sl[e] : -INFINITY;
+      s[2 + e] = ok ? s[2 + e] + sl[2 + e] : -INFINITY;
+      x0 = fmaxf(x0, s[e]);
+      x1 = fmaxf(x1, s[2 + e]);
+    }
 #pragma unroll
     for (int x = 1; x < 4; x <<= 1) {
       x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, x));
@@ -558,21 +566,23 @@ __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentS
     }
     if (t == 0) { mx_s[warp][g] = x0; mx_s[warp][g + 8] = x1; }
     __syncthreads();
-    const float n0 = fmaxf(m0, fmaxf(fmaxf(mx_s[0][g], mx_s[1][g]), fmaxf(mx_s[2][g], mx_s[3][g])));
-    const float n1 = fmaxf(m1, fmaxf(fmaxf(mx_s[0][g + 8], mx_s[1][g + 8]), fmaxf(mx_s[2][g + 8], mx_s[3][g + 8])));
+    float n0 = m0, n1 = m1;
+#pragma unroll
+    for (int w = 0; w < LAS_WARPS; ++w) {
+      n0 = fmaxf(n0, mx_s[w][g]);
+      n1 = fmaxf(n1, mx_s[w][g + 8]);
+    }
     const float f0 = expf(m0 - n0), f1 = expf(m1 - n1);  // every tile has a key, so n is finite
     m0 = n0; m1 = n1;
     float y0 = 0.f, y1 = 0.f;
 #pragma unroll
-    for (int i = 0; i < 2; ++i)
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int k = warp * 16 + 8 * i + 2 * t + e;
-        const float w0 = expf(s[i][e] - n0), w1 = expf(s[i][2 + e] - n1);
-        y0 += w0; y1 += w1;
-        split_bf16(w0, Ph[g * PS + k], Pl[g * PS + k]);
-        split_bf16(w1, Ph[(g + 8) * PS + k], Pl[(g + 8) * PS + k]);
-      }
+    for (int e = 0; e < 2; ++e) {
+      const int k = warp * 8 + 2 * t + e;
+      const float w0 = expf(s[e] - n0), w1 = expf(s[2 + e] - n1);
+      y0 += w0; y1 += w1;
+      split_bf16(w0, Ph[g * PS + k], Pl[g * PS + k]);
+      split_bf16(w1, Ph[(g + 8) * PS + k], Pl[(g + 8) * PS + k]);
+    }
     l0 = l0 * f0 + y0; l1 = l1 * f1 + y1;  // this thread's share; shares of lanes and warps are added at the end
 #pragma unroll
     for (int i = 0; i < TW; ++i) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
@@ -586,7 +596,7 @@ __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentS
       pfa_ldm4(al, Pl + aoff);
 #pragma unroll
       for (int i = 0; i < TW / 2; ++i) {
-        const int tile = 2 * (warp + 4 * i);
+        const int tile = 2 * (warp + LAS_WARPS * i);
         if (tile < tiles) {  // an odd last tile reads the row's next eight columns and drops them
           uint32_t vb[4];
           pfa_ldm4t(vb, Ks + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RS + tile * 8 + (lane >> 4) * 8);
@@ -610,12 +620,14 @@ __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentS
   if (tid < nh) {
     float* ml = p.part_ml + (row + (size_t)tid * p.nsplit) * 2;
     ml[0] = mx_s[0][tid];
-    ml[1] = k_begin < k_end ? sum_s[0][tid] + sum_s[1][tid] + sum_s[2][tid] + sum_s[3][tid] : 0.f;
+    float l = 0.f;
+    for (int w = 0; w < LAS_WARPS; ++w) l += sum_s[w][tid];
+    ml[1] = k_begin < k_end ? l : 0.f;
   }
   if (k_begin >= k_end) return;  // an empty run: its sum of zero makes the merge skip it
 #pragma unroll
   for (int i = 0; i < TW; ++i) {
-    const int tile = 2 * (warp + 4 * (i >> 1)) + (i & 1);
+    const int tile = 2 * (warp + LAS_WARPS * (i >> 1)) + (i & 1);
     if (tile < tiles) {
       const int c = 8 * tile + 2 * t;
       if (g < nh) *reinterpret_cast<float2*>(p.part_o + (row + (size_t)g * p.nsplit) * p.kvp + c) = make_float2(o[i][0], o[i][1]);
@@ -668,9 +680,11 @@ __global__ void __launch_bounds__(LAM_THREADS) latent_merge_kernel(const LatentD
   __syncthreads();
   for (int i = tid; i < p.kvp; i += LAM_THREADS) {
     float o = 0.f;
-#pragma unroll 8
-    for (int s = 0; s < p.nsplit; ++s)
-      if (w_s[s] > 0.f) o = fmaf(w_s[s], __ldcg(p.part_o + (base + s) * p.kvp + i), o);
+#pragma unroll 16
+    for (int s = 0; s < p.nsplit; ++s) {
+      const float v = __ldcg(p.part_o + (base + s) * p.kvp + i);
+      o = w_s[s] > 0.f ? fmaf(w_s[s], v, o) : o;  // an empty run's row was never written
+    }
     lam_s[i] = o;
   }
   __syncthreads();
@@ -704,7 +718,7 @@ __global__ void __launch_bounds__(LAM_THREADS) latent_merge_kernel(const LatentD
 }
 
 // ---- prompts -----------------------------------------------------------------------------------------------------
-constexpr int LAP_Q = 64, LAP_K = 64, LAP_THREADS = 128;
+constexpr int LAP_Q = 128, LAP_K = 64, LAP_THREADS = 256, LAP_WARPS = 8;
 
 struct LatentPrefillParams {
   const float* q;            // [T][q_stride], unrotated
@@ -725,13 +739,14 @@ struct LatentPrefillParams {
 };
 
 __host__ __device__ __forceinline__ int lap_qk_stride(int dim, int rot) { return (dim + rot + 15) / 16 * 16 + 8; }
+__host__ __device__ __forceinline__ int lap_value_cols(int vdim) { return vdim <= 32 ? 32 : vdim <= 64 ? 64 : vdim <= 128 ? 128 : 256; }
 __host__ __device__ __forceinline__ size_t lap_smem_bytes(int dim, int rot, int vp) {
   return ((size_t)(LAP_Q + LAP_K) * lap_qk_stride(dim, rot) + (size_t)LAP_K * (vp + 8)) * 2;
 }
 
 // grid = (query blocks of the longest run, heads, runs). VP = value columns per head rounded up to 32, 64, 128 or 256.
 template <int VP>
-__global__ void __launch_bounds__(LAP_THREADS) latent_prefill_kernel(const LatentPrefillParams p) {
+__global__ void __launch_bounds__(LAP_THREADS, VP <= 128 ? 2 : 1) latent_prefill_kernel(const LatentPrefillParams p) {
   extern __shared__ __align__(16) unsigned char lap_smem[];
   const RunDesc run = p.runs[blockIdx.z];
   const int q0 = blockIdx.x * LAP_Q, h = blockIdx.y;
@@ -743,15 +758,43 @@ __global__ void __launch_bounds__(LAP_THREADS) latent_prefill_kernel(const Laten
   __nv_bfloat16* Vs = Ks + LAP_K * QS;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int nq = min(LAP_Q, run.len - q0);
-  // queries: rotated, scaled into the base-2 exponent domain only after the product
-  for (int i = tid; i < LAP_Q * EP; i += LAP_THREADS) {
-    const int r = i / EP, c = i - r * EP;
-    float v = 0.f;
-    if (r < nq && c < E) {
-      const float* qr = p.q + (size_t)(run.row0 + q0 + r) * p.q_stride + h * E;
-      v = c < p.dim ? qr[c] : rotated(qr + p.dim, c - p.dim, p.rope + (size_t)(run.start + q0 + r) * p.pairs * 2, p.pairs);
+  const bool vec = !((p.dim | p.rot_dim | p.vdim | p.kv_stride | p.v_off | p.kr_stride | p.q_stride) & 7);
+  // queries, rotated; the scale is applied to the products
+  if (vec) {  // pieces of four elements (two pairs), eight of them in flight per thread
+    const int n4 = EP >> 2, d4 = p.dim >> 2, e4 = E >> 2;
+    for (int i0 = tid; i0 < LAP_Q * n4; i0 += 8 * LAP_THREADS) {
+      float4 v[8], cs[8];
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int i = i0 + k * LAP_THREADS, r = i / n4, c = i - r * n4;
+        const bool ok = r < nq && c < e4;
+        v[k] = ok ? *reinterpret_cast<const float4*>(p.q + (size_t)(run.row0 + q0 + r) * p.q_stride + h * E + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        cs[k] = make_float4(1.f, 0.f, 1.f, 0.f);  // pairs beyond the rotated ones pass
+        const int j = 2 * (c - d4);               // first of the piece's two pairs
+        if (ok && j >= 0) {
+          const float* table = p.rope + ((size_t)(run.start + q0 + r) * p.pairs + j) * 2;
+          if (j < p.pairs) { cs[k].x = table[0]; cs[k].y = table[1]; }
+          if (j + 1 < p.pairs) { cs[k].z = table[2]; cs[k].w = table[3]; }
+        }
+      }
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const int i = i0 + k * LAP_THREADS, r = i / n4, c = i - r * n4;
+        if (r < LAP_Q)
+          *reinterpret_cast<uint2*>(Qs + r * QS + 4 * c) = make_uint2(pack_bf2(v[k].x * cs[k].x - v[k].y * cs[k].y, v[k].y * cs[k].x + v[k].x * cs[k].y),
+                                                                      pack_bf2(v[k].z * cs[k].z - v[k].w * cs[k].w, v[k].w * cs[k].z + v[k].z * cs[k].w));
+      }
     }
-    Qs[r * QS + c] = __float2bfloat16(v);
+  } else {
+    for (int r = warp; r < LAP_Q; r += LAP_WARPS) {
+      const float* qr = p.q + (size_t)(run.row0 + q0 + min(r, nq - 1)) * p.q_stride + h * E;
+      const float* table = p.rope + (size_t)(run.start + q0 + min(r, nq - 1)) * p.pairs * 2;
+      for (int c = lane; c < EP; c += 32) {
+        float v = 0.f;
+        if (r < nq && c < E) v = c < p.dim ? qr[c] : rotated(qr + p.dim, c - p.dim, table, p.pairs);
+        Qs[r * QS + c] = __float2bfloat16(v);
+      }
+    }
   }
   const int qpos0 = run.start + q0;                       // position of the block's first query
   const int kfirst = p.window > 0 ? max(0, qpos0 - p.window + 1) : 0, klast = qpos0 + nq - 1;
@@ -763,41 +806,57 @@ __global__ void __launch_bounds__(LAP_THREADS) latent_prefill_kernel(const Laten
   for (int i = 0; i < NT_O; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   const float sc2 = p.scale * 1.4426950408889634f;
-  const bool vec = !((p.dim | p.rot_dim | p.vdim | p.kv_stride | p.v_off | p.kr_stride) & 7);
 
-  for (int kt = kfirst; kt <= klast; kt += LAP_K) {
+  // Key and value tiles have one buffer each: the next key tile is requested as soon as this one's scores are done, the
+  // next value tile after this one's products, so each copy runs under the other half of the work.
+  auto load_k = [&](int kt) {
     const int nk = min(LAP_K, klast - kt + 1);
-    __syncthreads();  // the previous tile (or the query tile's writers) are done
     const size_t crow = (size_t)(run.ctx0 + kt - base);
     if (vec) {
-      const int ce = EP >> 3, cd = p.dim >> 3, cn = E >> 3, cv = VP >> 3, cvn = p.vdim >> 3;
-      for (int i = tid; i < LAP_K * ce; i += LAP_THREADS) {
-        const int r = i / ce, c = i - r * ce;
-        __nv_bfloat16* d = Ks + r * QS + 8 * c;
-        if (r < nk && c < cn)
-          pfa_cp16(d, c < cd ? p.kv + (crow + r) * p.kv_stride + h * p.dim + 8 * c : p.kr + (crow + r) * p.kr_stride + 8 * (c - cd));
-        else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+      const int ce = EP >> 3, cd = p.dim >> 3, cn = E >> 3;
+      for (int r = warp; r < LAP_K; r += LAP_WARPS) {
+        const __nv_bfloat16* kv = p.kv + (crow + r) * p.kv_stride + h * p.dim;
+        const __nv_bfloat16* kr = p.kr + (crow + r) * p.kr_stride;
+        for (int c = lane; c < ce; c += 32) {
+          __nv_bfloat16* d = Ks + r * QS + 8 * c;
+          if (r < nk && c < cn) pfa_cp16(d, c < cd ? kv + 8 * c : kr + 8 * (c - cd));
+          else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
+        }
       }
-      for (int i = tid; i < LAP_K * cv; i += LAP_THREADS) {
-        const int r = i / cv, c = i - r * cv;
+    } else {
+      for (int i = tid; i < LAP_K * EP; i += LAP_THREADS) {
+        const int r = i / EP, c = i - r * EP;
+        __nv_bfloat16 v = __float2bfloat16(0.f);
+        if (r < nk && c < E) v = c < p.dim ? p.kv[(crow + r) * p.kv_stride + h * p.dim + c] : p.kr[(crow + r) * p.kr_stride + c - p.dim];
+        Ks[r * QS + c] = v;
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  auto load_v = [&](int kt) {
+    const int nk = min(LAP_K, klast - kt + 1);
+    const size_t crow = (size_t)(run.ctx0 + kt - base);
+    if (vec) {
+      constexpr int CV = VP >> 3;
+      const int cvn = p.vdim >> 3;
+      for (int i = tid; i < LAP_K * CV; i += LAP_THREADS) {
+        const int r = i / CV, c = i % CV;
         __nv_bfloat16* d = Vs + r * VS + 8 * c;
         if (r < nk && c < cvn) pfa_cp16(d, p.kv + (crow + r) * p.kv_stride + p.v_off + h * p.vdim + 8 * c);
         else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
       }
-      pfa_cp_wait_all();
     } else {
-      const __nv_bfloat16 zero = __float2bfloat16(0.f);
-      for (int i = tid; i < LAP_K * EP; i += LAP_THREADS) {
-        const int r = i / EP, c = i - r * EP;
-        __nv_bfloat16 v = zero;
-        if (r < nk && c < E) v = c < p.dim ? p.kv[(crow + r) * p.kv_stride + h * p.dim + c] : p.kr[(crow + r) * p.kr_stride + c - p.dim];
-        Ks[r * QS + c] = v;
-      }
       for (int i = tid; i < LAP_K * VP; i += LAP_THREADS) {
         const int r = i / VP, c = i - r * VP;
-        Vs[r * VS + c] = r < nk && c < p.vdim ? p.kv[(crow + r) * p.kv_stride + p.v_off + h * p.vdim + c] : zero;
+        Vs[r * VS + c] = r < nk && c < p.vdim ? p.kv[(crow + r) * p.kv_stride + p.v_off + h * p.vdim + c] : __float2bfloat16(0.f);
       }
     }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  load_k(kfirst);
+  load_v(kfirst);
+  for (int kt = kfirst; kt <= klast; kt += LAP_K) {
+    asm volatile("cp.async.wait_group 1;" ::: "memory");  // the key tile; its value tile may still be on its way
     __syncthreads();
     // scores: 16 queries x 64 keys per warp
     float s[8][4];
@@ -814,6 +873,9 @@ __global__ void __launch_bounds__(LAP_THREADS) latent_prefill_kernel(const Laten
         lap_mma(s[2 * nt + 1], a, kb[2], kb[3]);
       }
     }
+    __syncthreads();  // every warp has read the key tile
+    if (kt + LAP_K <= klast) load_k(kt + LAP_K);
+    else asm volatile("cp.async.commit_group;" ::: "memory");  // keeps one group per step
     float n0 = m0, n1 = m1;
 #pragma unroll
     for (int i = 0; i < 8; ++i) {
@@ -848,6 +910,8 @@ __global__ void __launch_bounds__(LAP_THREADS) latent_prefill_kernel(const Laten
         l1 += s[i][2 + e];
       }
     }
+    asm volatile("cp.async.wait_group 1;" ::: "memory");  // the value tile
+    __syncthreads();
     // weighted values
 #pragma unroll
     for (int kk = 0; kk < 4; ++kk) {
@@ -861,6 +925,9 @@ __global__ void __launch_bounds__(LAP_THREADS) latent_prefill_kernel(const Laten
         lap_mma(o[2 * nt + 1], a, vb[2], vb[3]);
       }
     }
+    __syncthreads();  // every warp has read the value tile
+    if (kt + LAP_K <= klast) load_v(kt + LAP_K);
+    else asm volatile("cp.async.commit_group;" ::: "memory");
   }
 #pragma unroll
   for (int x = 1; x < 4; x <<= 1) {

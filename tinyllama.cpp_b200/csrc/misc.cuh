@@ -20,6 +20,7 @@ __global__ void embed_kernel(const int* __restrict__ tokens, const float* __rest
 // token while a prompt is being replayed), positions[b] += 1, and the id is appended to the
 // step log. One block; warp w handles sequences w, w+nwarps, ...
 constexpr int PEN_WINDOW = 64;  // reference apply_repetition_penalty: window = 64 generated tokens
+constexpr int PEN_MAX_BATCH = 15;  // block models: most sequences of the penalised loop (it stays on the matvec path)
 
 struct SelectParams {
   const float* amax_val;  // [ranks][batch][parts_per_rank]

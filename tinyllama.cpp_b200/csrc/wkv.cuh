@@ -41,6 +41,12 @@ __global__ void __launch_bounds__(WKV_STEP_THREADS) wkv_step_kernel(const WkvSte
   __shared__ float r_s[WKV_MAX_DIM], k_s[WKV_MAX_DIM], w_s[WKV_MAX_DIM], part[WKV_STEP_THREADS], red[WKV_STEP_THREADS / 32];
   const int tid = threadIdx.x, h = blockIdx.x, b = blockIdx.y, D = p.dim, hc = h * D;
   pdl_launch_dependents();
+  constexpr int W2_KEEP = 8;  // pieces of the decay row requested ahead (rank up to 64)
+  const int rp = pad8(p.rank) >> 3;
+  const uint4* w2 = reinterpret_cast<const uint4*>(p.w2) + (size_t)(hc + min(tid, D - 1)) * rp;
+  uint4 wk[W2_KEEP];
+#pragma unroll
+  for (int i = 0; i < W2_KEEP; ++i) wk[i] = tid < D && i < rp ? ldg128(w2 + i) : make_uint4(0, 0, 0, 0);
   pdl_wait();
   const float* in = p.rkvg + (size_t)b * p.stride + hc;
   const int pos = p.positions[b];
@@ -63,11 +69,17 @@ __global__ void __launch_bounds__(WKV_STEP_THREADS) wkv_step_kernel(const WkvSte
   if (tid < D) {
     r_s[tid] = in[tid];
     k_s[tid] = in[p.off + tid];
-    float acc = p.w0[hc + tid];
-    const __nv_bfloat16* w2 = p.w2 + (size_t)(hc + tid) * pad8(p.rank);
     const float* low = p.low + (size_t)b * p.low_stride;
-#pragma unroll 8
-    for (int j = 0; j < p.rank; ++j) acc = fmaf(__bfloat162float(w2[j]), low[j], acc);
+    float acc = p.w0[hc + tid];
+    auto add = [&](const uint4& u, int i) {  // the row's padding is zero: elements beyond the rank only need to be finite
+      const float4 x = ld4_masked(low, 8 * i, p.rank), y = ld4_masked(low, 8 * i + 4, p.rank);
+      acc = fmaf(bf_lo(u.x), x.x, acc); acc = fmaf(bf_hi(u.x), x.y, acc); acc = fmaf(bf_lo(u.y), x.z, acc); acc = fmaf(bf_hi(u.y), x.w, acc);
+      acc = fmaf(bf_lo(u.z), y.x, acc); acc = fmaf(bf_hi(u.z), y.y, acc); acc = fmaf(bf_lo(u.w), y.z, acc); acc = fmaf(bf_hi(u.w), y.w, acc);
+    };
+#pragma unroll
+    for (int i = 0; i < W2_KEEP; ++i)
+      if (i < rp) add(wk[i], i);
+    for (int i = W2_KEEP; i < rp; ++i) add(ldg128(w2 + i), i);
     w_s[tid] = expf(-expf(acc));
   }
   __syncthreads();
@@ -103,6 +115,26 @@ constexpr int WKV_TILE = 16;  // tokens staged per step
 constexpr int WKV_KPT = 8;    // keys per thread
 constexpr int WKV_NC = 2;     // value columns per thread
 
+// two FP32 numbers in one 64-bit register pair; each half of an operation rounds like its scalar form
+typedef unsigned long long F2;
+__device__ __forceinline__ F2 f2(float lo, float hi) {
+  F2 r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+  return r;
+}
+__device__ __forceinline__ float f2_lo(F2 v) { return __uint_as_float((uint32_t)v); }
+__device__ __forceinline__ float f2_hi(F2 v) { return __uint_as_float((uint32_t)(v >> 32)); }
+__device__ __forceinline__ F2 fma2(F2 a, F2 b, F2 c) {
+  F2 r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ F2 mul2(F2 a, F2 b) {
+  F2 r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+
 struct WkvScanParams {
   const float* rkv;    // [T][stride]: r, k, v at offsets 0, off, 2 off
   int stride, off;
@@ -128,34 +160,38 @@ __host__ __device__ __forceinline__ int wkv_lanes(int dim) {
   return l;
 }
 __host__ __device__ __forceinline__ int wkv_cols(int dim) { return WKV_NC * WKV_SCAN_THREADS / wkv_lanes(dim); }
+// tiles in flight: four, or two where a token's row is long
+__host__ __device__ constexpr int wkv_stages(int lanes) { return lanes <= 16 ? 4 : 2; }
 __host__ __device__ __forceinline__ size_t wkv_scan_smem(int dim) {
-  return (size_t)2 * WKV_TILE * (3 * wkv_lanes(dim) * WKV_KPT + wkv_cols(dim)) * 4;
+  return (size_t)wkv_stages(wkv_lanes(dim)) * WKV_TILE * (3 * wkv_lanes(dim) * WKV_KPT + wkv_cols(dim)) * 4;
 }
 
 // grid = (column blocks of a head, heads, runs). L = lanes per column; a thread has two columns, COLS / 2 apart.
 template <int L>
 __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvScanParams p) {
-  extern __shared__ __align__(16) float scan_s[];  // two tiles of [token][r | k | w (DP each) | v (COLS)]
+  extern __shared__ __align__(16) float scan_s[];  // ring of tiles of [token][r | k | w (DP each) | v (COLS)]
   constexpr int DP = L * WKV_KPT, HALF = WKV_SCAN_THREADS / L, COLS = WKV_NC * HALF, ROW = 3 * DP + COLS;
   constexpr int G = L < WKV_TILE ? L : WKV_TILE;   // tokens whose outputs are reduced together
+  constexpr int STAGES = wkv_stages(L);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, D = p.dim, hc = h * D;
   const RunDesc run = p.runs[blockIdx.z];
   const int ln = tid % L, cl = tid / L, c0 = blockIdx.x * COLS;  // columns c0 + cl and c0 + cl + HALF
-  const int k0 = ln * WKV_KPT;
+  auto key = [&](int i) { return ln * 4 + (i & 3) + (i >> 2) * (DP / 2); };  // two runs of four keys: neighbouring lanes read neighbouring 16 bytes
   float* S = p.state + ((size_t)run.slot * p.heads + h) * D * D;
-  float st[WKV_NC][WKV_KPT], u[WKV_KPT];
+  F2 st[WKV_NC][WKV_KPT / 2], u[WKV_KPT / 2];  // pairs of neighbouring keys: packed FP32 arithmetic
 #pragma unroll
-  for (int i = 0; i < WKV_KPT; ++i) {
-    const int k = k0 + i;
-    u[i] = k < D ? p.u[hc + k] : 0.f;
+  for (int i = 0; i < WKV_KPT / 2; ++i) {
+    const int k = key(2 * i);
+    u[i] = f2(k < D ? p.u[hc + k] : 0.f, k + 1 < D ? p.u[hc + k + 1] : 0.f);
 #pragma unroll
     for (int n = 0; n < WKV_NC; ++n) {
       const int col = c0 + cl + n * HALF;
-      st[n][i] = run.start > 0 && k < D && col < D ? S[(size_t)k * D + col] : 0.f;
+      const bool ok = run.start > 0 && col < D;
+      st[n][i] = f2(ok && k < D ? S[(size_t)k * D + col] : 0.f, ok && k + 1 < D ? S[(size_t)(k + 1) * D + col] : 0.f);
     }
   }
-  // padding keys and columns stay zero in both tiles
-  for (int i = tid; i < 2 * WKV_TILE * ROW; i += WKV_SCAN_THREADS) scan_s[i] = 0.f;
+  // padding keys and columns stay zero in every tile of the ring
+  for (int i = tid; i < STAGES * WKV_TILE * ROW; i += WKV_SCAN_THREADS) scan_s[i] = 0.f;
   __syncthreads();
   const bool vec = !((D | hc | p.stride | p.off | p.decay_stride) & 3);  // 16-byte pieces possible
   const int nv = min(COLS, D - c0);
@@ -165,7 +201,7 @@ __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvSca
   auto fetch = [&](int tile) {  // a warp takes every fourth token of the tile
     const int first = tile * WKV_TILE, n = min(WKV_TILE, run.len - first);
     for (int t = warp; t < n; t += WKV_SCAN_THREADS / 32) {
-      float* d = scan_s + (size_t)((tile & 1) * WKV_TILE + t) * ROW;
+      float* d = scan_s + (size_t)((tile % STAGES) * WKV_TILE + t) * ROW;
       const size_t row = (size_t)(run.row0 + first + t);
       const float* rk = p.rkv + row * p.stride + hc;
       const float* dec = p.decay + row * p.decay_stride + hc;
@@ -186,12 +222,17 @@ __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvSca
     }
   };
   const int tiles = (run.len + WKV_TILE - 1) / WKV_TILE;
-  fetch(0);
+  auto commit = [] { asm volatile("cp.async.commit_group;" ::: "memory"); };
+  for (int i = 0; i < STAGES - 1; ++i) {  // one group per tile, empty ones beyond the last
+    if (i < tiles) fetch(i);
+    commit();
+  }
   for (int tile = 0; tile < tiles; ++tile) {
-    pfa_cp_wait_all();
-    __syncthreads();  // the tile has landed for everyone, and everyone has left the other buffer
-    if (tile + 1 < tiles) fetch(tile + 1);
-    const float* base = scan_s + (size_t)(tile & 1) * WKV_TILE * ROW;
+    asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
+    __syncthreads();  // the tile has landed for everyone, and everyone has left the one that is refilled now
+    if (tile + STAGES - 1 < tiles) fetch(tile + STAGES - 1);
+    commit();
+    const float* base = scan_s + (size_t)(tile % STAGES) * WKV_TILE * ROW;
     const int n = min(WKV_TILE, run.len - tile * WKV_TILE);
     auto group = [&](int g0, auto whole) {  // tokens g0 .. g0 + G - 1 of the tile
       float o[WKV_NC][G];
@@ -201,24 +242,26 @@ __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvSca
         for (int c = 0; c < WKV_NC; ++c) o[c][j] = 0.f;
         if (!decltype(whole)::value && g0 + j >= n) continue;
         const float* row = base + (g0 + j) * ROW;
-        const float4 r0 = *reinterpret_cast<const float4*>(row + k0), r1 = *reinterpret_cast<const float4*>(row + k0 + 4);
-        const float4 a0 = *reinterpret_cast<const float4*>(row + DP + k0), a1 = *reinterpret_cast<const float4*>(row + DP + k0 + 4);
-        const float4 w0 = *reinterpret_cast<const float4*>(row + 2 * DP + k0), w1 = *reinterpret_cast<const float4*>(row + 2 * DP + k0 + 4);
-        const float r[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
-        const float k[8] = {a0.x, a0.y, a0.z, a0.w, a1.x, a1.y, a1.z, a1.w};
-        const float w[8] = {w0.x, w0.y, w0.z, w0.w, w1.x, w1.y, w1.z, w1.w};
+        auto pairs = [&](const float* src, F2 (&v)[4]) {
+          const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(src + ln * 4), b = *reinterpret_cast<const ulonglong2*>(src + DP / 2 + ln * 4);
+          v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+        };
+        F2 r[4], k[4], w[4];
+        pairs(row, r);
+        pairs(row + DP, k);
+        pairs(row + 2 * DP, w);
 #pragma unroll
         for (int c = 0; c < WKV_NC; ++c) {
-          const float v = row[3 * DP + cl + c * HALF];
-          float x = 0.f, y = 0.f;  // two chains
+          const float v1 = row[3 * DP + cl + c * HALF];
+          const F2 v = f2(v1, v1);
+          F2 acc = f2(0.f, 0.f);
 #pragma unroll
-          for (int i = 0; i < WKV_KPT; ++i) {
-            const float kv = k[i] * v;
-            float& acc = i & 1 ? y : x;
-            acc = fmaf(r[i], fmaf(u[i], kv, st[c][i]), acc);
-            st[c][i] = fmaf(w[i], st[c][i], kv);
+          for (int i = 0; i < WKV_KPT / 2; ++i) {
+            const F2 kv = mul2(k[i], v);
+            acc = fma2(r[i], fma2(u[i], kv, st[c][i]), acc);
+            st[c][i] = fma2(w[i], st[c][i], kv);
           }
-          o[c][j] = x + y;
+          o[c][j] = f2_lo(acc) + f2_hi(acc);
         }
       }
       // sums over the column's lanes; lane j (mod G) ends up with token j
@@ -249,8 +292,11 @@ __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvSca
     const int col = c0 + cl + n * HALF;
     if (col < D)
 #pragma unroll
-      for (int i = 0; i < WKV_KPT; ++i)
-        if (k0 + i < D) S[(size_t)(k0 + i) * D + col] = st[n][i];
+      for (int i = 0; i < WKV_KPT / 2; ++i) {
+        const int k = key(2 * i);
+        if (k < D) S[(size_t)k * D + col] = f2_lo(st[n][i]);
+        if (k + 1 < D) S[(size_t)(k + 1) * D + col] = f2_hi(st[n][i]);
+      }
   }
   if (blockIdx.x == 0) {  // the heads' first blocks share the copy of the last token's h
     const float* src = p.h + (size_t)(run.row0 + run.len - 1) * p.h_stride;
