@@ -35,6 +35,9 @@ CONFIGS = {
     "aligned": config([latent(heads=4, dim=64, rot_dim=32, vdim=128, q_rank=96, kv_rank=128, window=50, rot={"base": 5000.0, "dims": 32}, ff=192, scale=0.15),
                        wkv(heads=2, dim=64, rank=16, ff=320)], width=192, vocab=256, loop={"start": 0, "stop": 2, "times": 2}),
     "wkv_only": config([wkv(heads=2, dim=128, rank=9), wkv(heads=5, dim=7, rank=1, ff=0), wkv(heads=1, dim=160, rank=24)], width=88),
+    # odd head dimensions; a window wider than the context; seventeen heads (one more than a group of the decode kernel)
+    "wide_window": config([latent(heads=17, dim=7, rot_dim=5, vdim=3, q_rank=9, kv_rank=19, window=5000, rot={"base": 31.0, "dims": 2}), wkv(heads=2, dim=33, rank=70)],
+                          width=65, vocab=77),
     "window_1": config([latent(window=1), latent(window=2, rot={"base": 50.0, "dims": 4})], loop={"start": 0, "stop": 1, "times": 2}),
 }
 

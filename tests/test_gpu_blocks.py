@@ -242,10 +242,10 @@ def test_slots_that_are_freed_and_used_again(pkg, case, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("batch", [2, 3, 7, 19])
+@pytest.mark.parametrize("batch", [2, 4, 7, 12, 19])
 def test_batches_of_unequal_requests_match_each_alone(pkg, case, dtype, batch):
-    """Prompts of unequal length in one call (runs share chunks), then joint decode steps in mixed slot order; 19 takes
-    the row path of large batches."""
+    """Prompts of unequal length in one call (runs share chunks), then joint decode steps in mixed slot order, on the
+    matvec path (small batches) and on the row path (large ones)."""
     c = case("odd")
     eng = engine(pkg, c, dtype, max_seqs=batch + 2)
     lens = [3 + 11 * i % 37 for i in range(batch)]

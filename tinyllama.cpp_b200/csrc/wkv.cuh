@@ -4,7 +4,7 @@
 //   wkv_step_kernel  one token of several sequences (decode): one block per (head, sequence); the decay's second matrix
 //                    product, the recurrence, the head norm and the gate in one launch
 //   wkv_scan_kernel  runs of tokens (prompts): the value columns of a head are independent of one another, so a block
-//                    takes a few columns of one head, keeps their state in registers (eight keys per thread) and walks
+//                    takes a few columns of one head, keeps their state in registers (four or eight keys of two columns per thread) and walks
 //                    the run's tokens, whose r, k, w, v pieces arrive in shared memory a tile ahead (cp.async)
 //
 // State of a slot: [head][key][value]. A token at position 0 starts from zeros whatever the slot held before.
@@ -112,7 +112,6 @@ __global__ void __launch_bounds__(WKV_STEP_THREADS) wkv_step_kernel(const WkvSte
 
 constexpr int WKV_SCAN_THREADS = 128;
 constexpr int WKV_TILE = 16;  // tokens staged per step
-constexpr int WKV_KPT = 8;    // keys per thread
 constexpr int WKV_NC = 2;     // value columns per thread
 
 // two FP32 numbers in one 64-bit register pair; each half of an operation rounds like its scalar form
@@ -153,34 +152,35 @@ struct WkvScanParams {
   int shift_stride;
 };
 
-// lanes per value column: a power of two with lanes * WKV_KPT >= dim
+// keys per thread, and lanes per value column: a power of two up to 32 with lanes * keys >= dim
+__host__ __device__ __forceinline__ int wkv_keys(int dim) { return dim <= 128 ? 4 : 8; }
 __host__ __device__ __forceinline__ int wkv_lanes(int dim) {
   int l = 1;
-  while (l * WKV_KPT < dim) l *= 2;
+  while (l * wkv_keys(dim) < dim) l *= 2;
   return l;
 }
 __host__ __device__ __forceinline__ int wkv_cols(int dim) { return WKV_NC * WKV_SCAN_THREADS / wkv_lanes(dim); }
 // tiles in flight: four, or two where a token's row is long
-__host__ __device__ constexpr int wkv_stages(int lanes) { return lanes <= 16 ? 4 : 2; }
+__host__ __device__ constexpr int wkv_stages(int row_keys) { return row_keys <= 128 ? 4 : 2; }
 __host__ __device__ __forceinline__ size_t wkv_scan_smem(int dim) {
-  return (size_t)wkv_stages(wkv_lanes(dim)) * WKV_TILE * (3 * wkv_lanes(dim) * WKV_KPT + wkv_cols(dim)) * 4;
+  return (size_t)wkv_stages(wkv_lanes(dim) * wkv_keys(dim)) * WKV_TILE * (3 * wkv_lanes(dim) * wkv_keys(dim) + wkv_cols(dim)) * 4;
 }
 
-// grid = (column blocks of a head, heads, runs). L = lanes per column; a thread has two columns, COLS / 2 apart.
-template <int L>
+// grid = (column blocks of a head, heads, runs). L = lanes per column, KPT = keys per thread; a thread has two columns, COLS / 2 apart.
+template <int L, int KPT>
 __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvScanParams p) {
   extern __shared__ __align__(16) float scan_s[];  // ring of tiles of [token][r | k | w (DP each) | v (COLS)]
-  constexpr int DP = L * WKV_KPT, HALF = WKV_SCAN_THREADS / L, COLS = WKV_NC * HALF, ROW = 3 * DP + COLS;
+  constexpr int DP = L * KPT, HALF = WKV_SCAN_THREADS / L, COLS = WKV_NC * HALF, ROW = 3 * DP + COLS;
   constexpr int G = L < WKV_TILE ? L : WKV_TILE;   // tokens whose outputs are reduced together
-  constexpr int STAGES = wkv_stages(L);
+  constexpr int STAGES = wkv_stages(DP);
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, D = p.dim, hc = h * D;
   const RunDesc run = p.runs[blockIdx.z];
   const int ln = tid % L, cl = tid / L, c0 = blockIdx.x * COLS;  // columns c0 + cl and c0 + cl + HALF
-  auto key = [&](int i) { return ln * 4 + (i & 3) + (i >> 2) * (DP / 2); };  // two runs of four keys: neighbouring lanes read neighbouring 16 bytes
+  auto key = [&](int i) { return ln * 4 + (i & 3) + (i >> 2) * (DP / 2); };  // runs of four keys: neighbouring lanes read neighbouring 16 bytes
   float* S = p.state + ((size_t)run.slot * p.heads + h) * D * D;
-  F2 st[WKV_NC][WKV_KPT / 2], u[WKV_KPT / 2];  // pairs of neighbouring keys: packed FP32 arithmetic
+  F2 st[WKV_NC][KPT / 2], u[KPT / 2];  // pairs of neighbouring keys: packed FP32 arithmetic
 #pragma unroll
-  for (int i = 0; i < WKV_KPT / 2; ++i) {
+  for (int i = 0; i < KPT / 2; ++i) {
     const int k = key(2 * i);
     u[i] = f2(k < D ? p.u[hc + k] : 0.f, k + 1 < D ? p.u[hc + k + 1] : 0.f);
 #pragma unroll
@@ -242,11 +242,14 @@ __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvSca
         for (int c = 0; c < WKV_NC; ++c) o[c][j] = 0.f;
         if (!decltype(whole)::value && g0 + j >= n) continue;
         const float* row = base + (g0 + j) * ROW;
-        auto pairs = [&](const float* src, F2 (&v)[4]) {
-          const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(src + ln * 4), b = *reinterpret_cast<const ulonglong2*>(src + DP / 2 + ln * 4);
-          v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
+        auto pairs = [&](const float* src, F2 (&v)[KPT / 2]) {
+#pragma unroll
+          for (int i = 0; i < KPT / 4; ++i) {
+            const ulonglong2 a = *reinterpret_cast<const ulonglong2*>(src + i * (DP / 2) + ln * 4);
+            v[2 * i] = a.x; v[2 * i + 1] = a.y;
+          }
         };
-        F2 r[4], k[4], w[4];
+        F2 r[KPT / 2], k[KPT / 2], w[KPT / 2];
         pairs(row, r);
         pairs(row + DP, k);
         pairs(row + 2 * DP, w);
@@ -256,7 +259,7 @@ __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvSca
           const F2 v = f2(v1, v1);
           F2 acc = f2(0.f, 0.f);
 #pragma unroll
-          for (int i = 0; i < WKV_KPT / 2; ++i) {
+          for (int i = 0; i < KPT / 2; ++i) {
             const F2 kv = mul2(k[i], v);
             acc = fma2(r[i], fma2(u[i], kv, st[c][i]), acc);
             st[c][i] = fma2(w[i], st[c][i], kv);
@@ -292,7 +295,7 @@ __global__ void __launch_bounds__(WKV_SCAN_THREADS) wkv_scan_kernel(const WkvSca
     const int col = c0 + cl + n * HALF;
     if (col < D)
 #pragma unroll
-      for (int i = 0; i < WKV_KPT / 2; ++i) {
+      for (int i = 0; i < KPT / 2; ++i) {
         const int k = key(2 * i);
         if (k < D) S[(size_t)k * D + col] = f2_lo(st[n][i]);
         if (k + 1 < D) S[(size_t)(k + 1) * D + col] = f2_hi(st[n][i]);
