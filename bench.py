@@ -333,7 +333,7 @@ def run_block(args):
     result = {"block model": throughput(block, "bf16, bf16 latent cache, window %d" % shape["window"]), "packed model": throughput(packed, "Q8_0, INT8 KV cache")}
     progress("throughput done")
     kernels = {}
-    for label, b, rows in (("decode batch 1", 1, False), ("decode batch 8", 8, False), (f"prompt chunk of {chunk}", 1, True)):
+    for label, b, rows in (("decode batch 1", 1, False), ("decode batch 4", 4, False), (f"prompt chunk of {chunk}", 1, True)):
         eng = block(b, 4096)
         kernels[label] = {}
         for which, (name, flops) in block_kinds(shape, b, rows, chunk, 4096).items():
