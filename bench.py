@@ -236,7 +236,7 @@ def parity_in_run(eng, shape, scheme, kv):
             "logit_gate_note": None if not tag.endswith("i8") else "INT8 cache: 2e-2 or a quarter of the oracle's own INT8-vs-FP32 drift (rounding flips of cached values)"}
 
 
-def block_kinds(shape, batch, rows, chunk, context, act_bytes=4):
+def block_kinds(shape, batch, rows, chunk, context):
     """FLOPs of each timed kind of a block model's launch (selector -> name, FLOPs per launch)."""
     s = shape
     H, D, R, V, W = s["heads"], s["dim"], s["rot_dim"], s["vdim"], s["width"]
@@ -286,7 +286,6 @@ def run_block(args):
             eng = load(b, prompt_len + 2 * warmup + 2 * steps + 8 if b == 1 else 1024 + 2 * warmup + steps + 8)
             n = prompt_len if b == 1 else 1024
             prompts_b = [rng.integers(0, shape["vocab"], n).astype(np.int32) for _ in range(b)]
-            first = []
             for i, p in enumerate(prompts_b):
                 eng.prefill(p[:16], slot=i)
                 eng.kv_reset(i)
@@ -299,7 +298,7 @@ def run_block(args):
                         best = min(best, time.perf_counter() - t0)
                     out["prompt"][f"{m} tokens"] = {"tokens_per_s": round(m / best), "ms": round(best * 1e3, 3)}
             first = eng.prefill_batch(prompts_b).argmax(axis=1)
-            _, _ = eng.generate_greedy(first, [n] * b, warmup)
+            eng.generate_greedy(first, [n] * b, warmup)
             _, ms = eng.generate_greedy(first, [n + warmup] * b, steps)
             st = eng.stats()
             ctx = n + warmup + steps / 2
