@@ -216,7 +216,9 @@ int b200_engine_stats(const b200_engine* e, int64_t* kernel_launches_per_step, i
 /* Repeats one kernel of the decode step (or, with 16 added to the selector, of the batch / prompt path) alone `iters` times over
  * distinct layers' weights and returns its mean CUDA-event duration and algorithmic bytes. 0 = gate/up, 1 = first projections,
  * 2 = O projection, 3 = down projection, 4 = lm_head, 5 = attention; block models: 5 = query projection, 6 = latent attention,
- * 7 = WKV projections, 8 = WKV recurrence, and of a prompt chunk also 9 = key / value expansion, 10 = cache append, 11 = row norm
+ * 7 = WKV projections, 8 = WKV recurrence, and of a prompt chunk also 9 = key / value expansion, 10 = cache append, 11 = row norm;
+ * 32 = projections, 33 = attention of a shared-kv attention layer (34 = its cache append), 35 = projections, 36 = recurrence of an
+ * RG-LRU layer (of a prompt chunk 36 = gates and recurrence inside tiles, 37 = across tiles and output product)
  * (their slots are cleared afterwards). */
 int b200_engine_time_kernel(b200_engine* e, int which, int iters, float* mean_us, int64_t* bytes_per_launch);
 

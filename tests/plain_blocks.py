@@ -152,9 +152,88 @@ def wkv(h, W, m, eps, state=None, rnd=exact):
     return rnd(o.reshape(T, H * D) * W("norm") * gate) @ W("o").T, (h[-1], S)
 
 
+def softcap(z, cap):
+    return z if not cap else cap * np.tanh(z / cap)
+
+
+def seen_keys(p, mask):
+    """First key position that the query at position p sees, by a chunked mask (blocks of `size` positions)."""
+    return p // mask["size"] * mask["size"] if mask else 0
+
+
+def sink_weights(s):
+    """Softmax over the last axis with one more term, exp(0), in the denominator."""
+    top = np.maximum(s.max(axis=-1, keepdims=True), 0.0)
+    e = np.exp(s - top)
+    return e / (np.exp(-top) + e.sum(axis=-1, keepdims=True))
+
+
+def shared_kv_attention(h, W, m, start=0, cache=None, rnd=exact):
+    """Grouped-query attention whose values are its unrotated keys; chunked mask, capped scores, sink. cache: (unrotated keys,
+    rotated keys) of the positions before `start`, each [positions][kv_heads][dim]. Returns (output, new cache)."""
+    T, H, G, D = len(h), m["heads"], m["kv_heads"], m["dim"]
+    pos = np.arange(start, start + T)
+    h = rnd(h)
+    q = rnd(rotate((h @ W("q").T).reshape(T, H, D), pos, m["rot"]))
+    raw = (h @ W("k").T).reshape(T, G, D)
+    v, k = rnd(raw), rnd(rotate(raw, pos, m["rot"]))
+    if cache is not None:
+        v, k = np.concatenate([cache[0], v]), np.concatenate([cache[1], k])
+    out = np.empty((T, H, D))
+    for t in range(T):
+        p = start + t
+        lo = seen_keys(p, m.get("mask"))
+        for x in range(H):
+            g = x // (H // G)
+            s = softcap(k[lo:p + 1, g] @ q[t, x] * m["scale"], m.get("softcap"))
+            out[t, x] = rnd(sink_weights(s)) @ v[lo:p + 1, g]
+    return rnd(out.reshape(T, H * D)) @ W("o").T, (v, k)
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1 + np.tanh(math.sqrt(2 / math.pi) * (z + 0.044715 * z ** 3)))
+
+
+def causal_conv(x, w, b, before):
+    """x [T][channels]; w [channels][taps], last column = the current token; before [taps - 1][channels] = earlier inputs."""
+    taps = w.shape[1]
+    full = np.concatenate([before, x])
+    return sum(full[k:k + len(x)] * w[:, k] for k in range(taps)) + b, full[len(full) - taps + 1:]
+
+
+def gated_recurrence(u, r, i, lam, S):
+    """Per channel: a = exp(-8 r softplus(lam)), S <- a S + sqrt(1 - a^2) i u. All [T][channels]. Returns (S of every token, S after)."""
+    log_a = -8.0 * r * np.logaddexp(0.0, lam)
+    a, x = np.exp(log_a), np.sqrt(-np.expm1(2 * log_a)) * i * u
+    out = np.empty_like(u)
+    for t in range(len(u)):
+        S = a[t] * S + x[t]
+        out[t] = S
+    return out, S
+
+
+def rglru(h, W, m, state=None, rnd=exact):
+    """state: (last taps - 1 inputs of the convolution, S). Returns (output, new state)."""
+    T, N, B = len(h), m["width"], m["blocks"]
+    before, S = state if state is not None else (np.zeros((m["conv"] - 1, N)), np.zeros(N))
+    h = rnd(h)
+    y = gelu_tanh(h @ W("y").T + W("y.b"))
+    u, before = causal_conv(h @ W("x").T + W("x.b"), W("conv"), W("conv.b"), before)
+    ub = u.reshape(T, B, N // B)
+    r = sigmoid(np.einsum("boi,tbi->tbo", W("ra"), ub) + W("ra.b")).reshape(T, N)
+    i = sigmoid(np.einsum("boi,tbi->tbo", W("ri"), ub) + W("ri.b")).reshape(T, N)
+    out, S = gated_recurrence(u, r, i, W("lam"), S)
+    return rnd(out * y) @ W("o").T, (before, S)
+
+
 def dense_relu(h, W, rnd=exact):
     h = rnd(h)
     return rnd(np.maximum(h @ W("gate").T, 0) * (h @ W("up").T)) @ W("down").T
+
+
+def dense_silu(h, W, rnd=exact):
+    h = rnd(h)
+    return rnd(silu(h @ W("gate").T) * (h @ W("up").T)) @ W("down").T
 
 
 # ---- model -------------------------------------------------------------------------------------------------------
@@ -167,6 +246,9 @@ def layer_runs(cfg):
 
 
 class PlainModel:
+    """Nezolix (each sublayer normalised before and after, own head) or Pizilix (normalised before, norm weights stored around
+    zero, embedding added again before every further pass of a loop, tied and capped head)."""
+
     def __init__(self, cfg, tensors, rnd=exact):
         self.rnd = rnd
         self.cfg, self.t = cfg, {k: np.asarray(v, np.float64) for k, v in tensors.items()}
@@ -177,8 +259,13 @@ class PlainModel:
 
     def run(self, tokens, trace=None):
         """The next tokens of the sequence; returns their logits [T][vocab]."""
+        x = (self.run_pizilix if self.cfg["architecture"] == "Pizilix" else self.run_nezolix)(np.asarray(tokens), trace)
+        self.pos += len(x)
+        return x
+
+    def run_nezolix(self, tokens, trace):
         cfg, eps = self.cfg, self.cfg["norm"]["eps"]
-        x = self.t["embed"][np.asarray(tokens)] * cfg["embedding"]["scale"]
+        x = self.t["embed"][tokens] * cfg["embedding"]["scale"]
         for i, l in enumerate(layer_runs(cfg)):
             lay = cfg["layers"][l]
             N = lambda s: self.t[f"l{l}.{s}"]
@@ -194,8 +281,29 @@ class PlainModel:
                 x = x + rms(y, N("norm2b"), eps)
             if trace is not None:
                 trace.append(x.copy())
-        self.pos += len(x)
         return self.rnd(rms(x, self.t["final.norm"], eps)) @ self.t["head"].T
+
+    def run_pizilix(self, tokens, trace):
+        cfg, eps = self.cfg, self.cfg["norm"]["eps"]
+        x = first = self.t["embed"][tokens]
+        runs, loop = layer_runs(cfg), cfg.get("loop")
+        again = {loop["start"] + n * (loop["stop"] - loop["start"]) for n in range(1, loop["times"])} if loop else set()
+        for i, l in enumerate(runs):
+            lay = cfg["layers"][l]
+            W = lambda s: self.t[f"l{l}.mix.{s}"]
+            norm = lambda s: rms(x, 1 + self.t[f"l{l}.{s}"], eps)
+            if i in again:
+                x = x + first
+            if lay["type"] == "rglru":
+                y, self.state[i] = rglru(norm("norm1"), W, lay["mixer"], self.state[i], self.rnd)
+            else:
+                y, self.state[i] = shared_kv_attention(norm("norm1"), W, lay["mixer"], self.pos, self.state[i], self.rnd)
+            x = x + y
+            if lay.get("mlp"):
+                x = x + dense_silu(norm("norm2"), lambda s: self.t[f"l{l}.mlp.{s}"], self.rnd)
+            if trace is not None:
+                trace.append(x.copy())
+        return softcap(self.rnd(rms(x, 1 + self.t["final.norm"], eps)) @ self.t["embed"].T, cfg.get("logit_softcap"))
 
 
 def greedy(cfg, tensors, prompt, steps):

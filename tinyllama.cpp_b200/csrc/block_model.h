@@ -25,16 +25,23 @@ struct BlockLayer {
   // wkv
   DenseW r, k, v, wg, w1, w2;
   float *mu[5] = {nullptr}, *w0 = nullptr, *u = nullptr, *norm = nullptr;
+  // shared-kv attention (keys: k)
+  DenseW q;
+  // rg-lru: the two branches, the gate matrices as [width][block size], the convolution as [taps][padded width]
+  DenseW in_y, in_x, ra, ri;
+  float *y_b = nullptr, *x_b = nullptr, *ra_b = nullptr, *ri_b = nullptr, *conv = nullptr, *conv_b = nullptr, *decay = nullptr;
 };
 
 // What one layer run keeps per sequence slot (a looped layer has one of these per pass).
 struct BlockRun {
   int layer = 0;
-  void* cache = nullptr;   // latent attention: ring of rows [slot][cap][crow]
+  bool add_embedding = false;  // the embedding output joins the stream ahead of this run
+  void* cache = nullptr;   // latent attention: ring of rows [slot][cap][crow]; shared-kv attention: [slot][kv_heads][cap][crow]
   int cap = 0, crow = 0, kvp = 0;
   size_t cache_slot_bytes = 0;
-  float* state = nullptr;  // wkv: [slot][heads][dim][dim]
-  float* shift = nullptr;  // wkv: [slot][2][padded width], the previous token's input by position parity
+  float* state = nullptr;  // wkv: [slot][heads][dim][dim]; rg-lru: [slot][padded width]
+  float* shift = nullptr;  // wkv: [slot][2][padded model width], the previous token's input by position parity; rg-lru: [slot][taps][padded width], the convolution's last inputs
+  size_t state_slot = 0, shift_slot = 0;  // floats per slot
 };
 
 struct BlockModel {
@@ -43,7 +50,8 @@ struct BlockModel {
   std::vector<int> order;  // layer of every run
   std::vector<BlockLayer> layers;
   std::vector<BlockRun> runs;
-  DenseW embed, head;
+  DenseW embed, head;      // head: the embedding table itself when they are tied
+  float* first = nullptr;  // embedding output of the rows in work, kept for a loop that adds it again
   float* final_norm = nullptr;
   int Wp = 0;              // padded width
   int chunk = 1024;        // prompt tokens per chunk

@@ -19,12 +19,16 @@ __device__ __forceinline__ float to_operand<float>(float v) { return v; }
 template <>
 __device__ __forceinline__ __nv_bfloat16 to_operand<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
 
-// x[b][:] = table[tokens[b]][:] * scale. grid.x = tokens.
+// x[b][:] = table[tokens[b]][:] * scale, and the same into `again` if given. grid.x = tokens.
 __global__ void embed_bf16_kernel(const int* __restrict__ tokens, const __nv_bfloat16* __restrict__ table, int ld, float scale, float* __restrict__ x,
-                                  int x_stride, int W, int vocab) {
+                                  float* __restrict__ again, int x_stride, int W, int vocab) {
   const int b = blockIdx.x;
   const int tok = min(max(tokens[b], 0), vocab - 1);
-  for (int i = threadIdx.x; i < W; i += blockDim.x) x[(size_t)b * x_stride + i] = __bfloat162float(table[(size_t)tok * ld + i]) * scale;
+  for (int i = threadIdx.x; i < W; i += blockDim.x) {
+    const float v = __bfloat162float(table[(size_t)tok * ld + i]) * scale;
+    x[(size_t)b * x_stride + i] = v;
+    if (again) again[(size_t)b * x_stride + i] = v;
+  }
 }
 
 constexpr int ROW_THREADS = 256;
@@ -33,7 +37,8 @@ struct NormRowsParams {
   float* x;            // [T][x_stride] residual stream, updated in place when `add` is given
   int x_stride, W;
   const float* add;    // pending sublayer output [T][x_stride]
-  const float* add_w;
+  const float* add_w;  // its norm, or nullptr: added as it is
+  const float* add2;   // further rows added to the stream [T][x_stride] (only with add), or nullptr
   const float* norm_w; // nullptr: only the residual update
   float eps;
   const int* gather;   // row i of the output comes from row gather[i] of x (x itself is left as it is then)
@@ -42,7 +47,7 @@ struct NormRowsParams {
   int out_stride;
 };
 
-// One block per row: x += rms(add) * add_w; out = rms(x) * norm_w.
+// One block per row: x += rms(add) * add_w (or add), x += add2; out = rms(x) * norm_w.
 template <typename A>
 __global__ void __launch_bounds__(ROW_THREADS) norm_rows_kernel(const NormRowsParams p) {
   extern __shared__ __align__(16) float row_s[];
@@ -53,7 +58,7 @@ __global__ void __launch_bounds__(ROW_THREADS) norm_rows_kernel(const NormRowsPa
   float4* s4 = reinterpret_cast<float4*>(row_s);
   float f = 0.f, ss[1];
   const float* ar = p.add ? p.add + src * p.x_stride : nullptr;
-  if (ar) {
+  if (ar && p.add_w) {
     ss[0] = 0.f;
     for (int j = tid; j < n4; j += ROW_THREADS) {
       const float4 a = ld4_masked(ar, 4 * j, p.W);
@@ -67,8 +72,17 @@ __global__ void __launch_bounds__(ROW_THREADS) norm_rows_kernel(const NormRowsPa
   for (int j = tid; j < n4; j += ROW_THREADS) {
     float4 v = ld4_masked(xr, 4 * j, p.W);
     if (ar) {
-      const float4 a = s4[j], w = ld4_masked(p.add_w, 4 * j, p.W);
-      v.x += a.x * f * w.x; v.y += a.y * f * w.y; v.z += a.z * f * w.z; v.w += a.w * f * w.w;
+      if (p.add_w) {
+        const float4 a = s4[j], w = ld4_masked(p.add_w, 4 * j, p.W);
+        v.x += a.x * f * w.x; v.y += a.y * f * w.y; v.z += a.z * f * w.z; v.w += a.w * f * w.w;
+      } else {
+        const float4 a = ld4_masked(ar, 4 * j, p.W);
+        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+      }
+      if (p.add2) {
+        const float4 e = ld4_masked(p.add2 + src * p.x_stride, 4 * j, p.W);
+        v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+      }
       if (!p.gather) *reinterpret_cast<float4*>(xr + 4 * j) = v;
     }
     s4[j] = v;

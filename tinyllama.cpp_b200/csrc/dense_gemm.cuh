@@ -27,13 +27,14 @@ struct DgmSeg {
   const __nv_bfloat16* w;  // [rows][pad8(K)]
   const void* x;           // [T][x_ld] bfloat16 (sgemm: FP32)
   int x_ld;
-  int rows;                // matrix rows (ACT_RELU_GLU: interleaved gate and up rows)
+  int rows;                // matrix rows (gated products: interleaved gate and up rows)
   int outs;                // outputs (= rows, or the inner size of the gated product)
   int act;
   void* y;                 // [T][y_stride], FP32 or bfloat16
   int y_stride;
   int y_bf16;
-  const float* aux;        // per-row bias of ACT_DECAY
+  const float* bias;       // [rows], or nullptr
+  float arg;               // cap of ACT_SOFTCAP
 };
 
 struct DgmParams {
@@ -86,15 +87,15 @@ __device__ __forceinline__ void dgm_put(__nv_bfloat16* y, float v) { *y = __floa
 
 // Sixteen columns (tokens t0 ..) of this lane's row: activation and store. ACT is a compile-time copy of sg.act.
 template <int ACT, typename Y>
-__device__ __forceinline__ void dgm_store16(const DgmSeg& sg, int row, int t0, int T, float aux, const float (&v)[16]) {
-  if (ACT == ACT_RELU_GLU) {
+__device__ __forceinline__ void dgm_store16(const DgmSeg& sg, int row, int t0, int T, float bias, const float (&v)[16]) {
+  if (act_is_glu(ACT)) {
     const int o = (row >> 4) * 8 + (row & 7);
     const bool mine = !(row & 8) && o < sg.outs;
     Y* y = static_cast<Y*>(sg.y) + (size_t)t0 * sg.y_stride + o;
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
       const float up = __shfl_sync(0xffffffffu, v[j], ((threadIdx.x & 31) & 23) + 8);
-      if (mine && t0 + j < T) dgm_put(y, fmaxf(v[j], 0.f) * up);
+      if (mine && t0 + j < T) dgm_put(y, glu_act(ACT, v[j], up));
       y += sg.y_stride;
     }
   } else if (row < sg.rows) {
@@ -102,20 +103,23 @@ __device__ __forceinline__ void dgm_store16(const DgmSeg& sg, int row, int t0, i
     const int n = min(16, T - t0);
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
-      if (j < n) dgm_put(y, dense_act(ACT, v[j], aux));
+      if (j < n) dgm_put(y, dense_act(ACT, v[j] + bias, sg.arg));
       y += sg.y_stride;
     }
   }
 }
 template <typename Y>
-__device__ __forceinline__ void dgm_store16(const DgmSeg& sg, int row, int t0, int T, float aux, const float (&v)[16]) {
+__device__ __forceinline__ void dgm_store16(const DgmSeg& sg, int row, int t0, int T, float bias, const float (&v)[16]) {
   switch (sg.act) {
-    case ACT_SIGMOID: dgm_store16<ACT_SIGMOID, Y>(sg, row, t0, T, aux, v); break;
-    case ACT_SILU: dgm_store16<ACT_SILU, Y>(sg, row, t0, T, aux, v); break;
-    case ACT_TANH: dgm_store16<ACT_TANH, Y>(sg, row, t0, T, aux, v); break;
-    case ACT_DECAY: dgm_store16<ACT_DECAY, Y>(sg, row, t0, T, aux, v); break;
-    case ACT_RELU_GLU: dgm_store16<ACT_RELU_GLU, Y>(sg, row, t0, T, aux, v); break;
-    default: dgm_store16<ACT_NONE, Y>(sg, row, t0, T, aux, v);
+    case ACT_SIGMOID: dgm_store16<ACT_SIGMOID, Y>(sg, row, t0, T, bias, v); break;
+    case ACT_SILU: dgm_store16<ACT_SILU, Y>(sg, row, t0, T, bias, v); break;
+    case ACT_TANH: dgm_store16<ACT_TANH, Y>(sg, row, t0, T, bias, v); break;
+    case ACT_DECAY: dgm_store16<ACT_DECAY, Y>(sg, row, t0, T, bias, v); break;
+    case ACT_GELU: dgm_store16<ACT_GELU, Y>(sg, row, t0, T, bias, v); break;
+    case ACT_SOFTCAP: dgm_store16<ACT_SOFTCAP, Y>(sg, row, t0, T, bias, v); break;
+    case ACT_SILU_GLU: dgm_store16<ACT_SILU_GLU, Y>(sg, row, t0, T, bias, v); break;
+    case ACT_RELU_GLU: dgm_store16<ACT_RELU_GLU, Y>(sg, row, t0, T, bias, v); break;
+    default: dgm_store16<ACT_NONE, Y>(sg, row, t0, T, bias, v);
   }
 }
 
@@ -210,9 +214,9 @@ __global__ void __launch_bounds__(DGM_THREADS, 1) dense_gemm_kernel(const DgmPar
   } else {
     // ---- epilogue warps: lanes 32 (w & 3) .. of the accumulator = weight rows, the two groups of four split the tokens ----
     const int r = 32 * (warp & 3) + lane, c_begin = (warp >> 2) * (p.NT / 2), c_end = c_begin + p.NT / 2;
-    auto store = [&](const DgmSeg& sg, int row, int t0, float aux, const float (&v)[16]) {
-      if (sg.y_bf16) dgm_store16<__nv_bfloat16>(sg, row, t0, p.T, aux, v);
-      else dgm_store16<float>(sg, row, t0, p.T, aux, v);
+    auto store = [&](const DgmSeg& sg, int row, int t0, float bias, const float (&v)[16]) {
+      if (sg.y_bf16) dgm_store16<__nv_bfloat16>(sg, row, t0, p.T, bias, v);
+      else dgm_store16<float>(sg, row, t0, p.T, bias, v);
     };
     int n = 0;
     for (int u = blockIdx.x; u < units; u += gridDim.x, ++n) {
@@ -233,7 +237,7 @@ __global__ void __launch_bounds__(DGM_THREADS, 1) dense_gemm_kernel(const DgmPar
       tc_fence_after();
       const DgmSeg& sg = p.seg[w.seg];
       const int row = w.row0 + r;
-      const float aux = sg.aux && row < sg.rows ? sg.aux[row] : 0.f;
+      const float bias = sg.bias && row < sg.rows ? sg.bias[row] : 0.f;
       const uint32_t base = tmem + ((uint32_t)(32 * (warp & 3)) << 16) + (uint32_t)(buf * p.acc_cols);
       float* part = p.ws + ((size_t)((w.k0 / p.ksteps) * p.tiles_m * p.tiles_n + w.tile) * p.NT) * TC_M + r;
       for (int c = c_begin; c < c_end && w.t0 + c < p.T; c += 16) {
@@ -243,7 +247,7 @@ __global__ void __launch_bounds__(DGM_THREADS, 1) dense_gemm_kernel(const DgmPar
 #pragma unroll
           for (int j = 0; j < 16; ++j) part[(size_t)(c + j) * TC_M] = v[j];
         } else {
-          store(sg, row, w.t0 + c, aux, v);
+          store(sg, row, w.t0 + c, bias, v);
         }
       }
       tc_fence_before();
@@ -268,7 +272,7 @@ __global__ void __launch_bounds__(DGM_THREADS, 1) dense_gemm_kernel(const DgmPar
             for (int z = 0; z < p.ksplit; ++z)
 #pragma unroll
               for (int j = 0; j < 16; ++j) v[j] += __ldcg(sum + z * step + (size_t)(c + j) * TC_M);
-            store(sg, row, w.t0 + c, aux, v);
+            store(sg, row, w.t0 + c, bias, v);
           }
         }
         asm volatile("bar.sync 1, %0;" ::"n"(32 * DGM_EPI_WARPS) : "memory");  // sh.last is read before the next unit writes it
@@ -292,7 +296,7 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const DgmParams p) {
   auto tiles = [&](int s) { return (p.seg[s].outs + 63) / 64; };
   while (seg + 1 < p.nseg && mt >= tiles(seg)) { mt -= tiles(seg); ++seg; }
   const DgmSeg& sg = p.seg[seg];
-  const bool glu = sg.act == ACT_RELU_GLU;
+  const bool glu = act_is_glu(sg.act);
   const int ld = pad8(p.K), r0 = mt * 64, t0 = blockIdx.y * 64;
   const int tr = tid & 15, tt = tid >> 4;
   float kept[4][4];  // the gated product keeps its gate half while the up half is computed
@@ -328,9 +332,9 @@ __global__ void __launch_bounds__(256) sgemm_kernel(const DgmParams p) {
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
         const int row = r0 + 4 * tr + i, t = t0 + 4 * tt + j;
-        if (glu && half == 0) { kept[i][j] = fmaxf(acc[i][j], 0.f); continue; }
+        if (glu && half == 0) { kept[i][j] = acc[i][j]; continue; }
         if (row >= sg.outs || t >= p.T) continue;
-        const float v = glu ? kept[i][j] * acc[i][j] : dense_act(sg.act, acc[i][j], sg.aux ? sg.aux[row] : 0.f);
+        const float v = glu ? glu_act(sg.act, kept[i][j], acc[i][j]) : dense_act(sg.act, acc[i][j] + (sg.bias ? sg.bias[row] : 0.f), sg.arg);
         if (sg.y_bf16) static_cast<__nv_bfloat16*>(sg.y)[(size_t)t * sg.y_stride + row] = __float2bfloat16(v);
         else static_cast<float*>(sg.y)[(size_t)t * sg.y_stride + row] = v;
       }

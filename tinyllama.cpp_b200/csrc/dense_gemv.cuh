@@ -1,12 +1,13 @@
 // Matvec over bfloat16 weights for decode batches of the block models, with the layer's row work fused in.
 //
 // Prologue (every CTA repeats it for the vectors it needs; one CTA stores what the rest of the step reads):
-//   1. the pending sublayer output is normalised and added to the residual stream: x <- x + rms(add) * add_w;
+//   1. the pending sublayer output is added to the residual stream, normalised if it has a norm of its own:
+//      x <- x + rms(add) * add_w, or x <- x + add; a looped stretch may then add its embedding rows once more;
 //   2. the stream is normalised for this launch: h = rms(x) * norm_w;
 //   3. token-shift launches mix h with the previous token's h, with one mix per segment: h + (h' - h) * mu_seg.
 // Each step is optional. Activations stay in FP32 in shared memory, weights are read once from HBM as 16-byte pieces
-// straight into registers, products and sums are FP32. Epilogue per segment: an activation, or the gated product
-// relu(gate) * up whose two rows one warp owns, or the logits with argmax partials and repetition penalty.
+// straight into registers, products and sums are FP32. Epilogue per segment: bias and activation, or the gated product
+// act(gate) * up whose two rows one warp owns, or the logits with argmax partials and repetition penalty.
 //
 // A warp owns two rows; K is walked in pieces of 8 elements per lane, four pieces of both rows in flight. The pieces
 // of a warp's first task are requested before the launch waits for the previous kernel (programmatic dependent launch):
@@ -19,19 +20,25 @@
 
 namespace b200 {
 
-enum : int { ACT_NONE = 0, ACT_SIGMOID, ACT_SILU, ACT_TANH, ACT_DECAY, ACT_RELU_GLU };
+enum : int { ACT_NONE = 0, ACT_SIGMOID, ACT_SILU, ACT_TANH, ACT_DECAY, ACT_GELU, ACT_SOFTCAP, ACT_RELU_GLU, ACT_SILU_GLU };
 
+__host__ __device__ __forceinline__ bool act_is_glu(int act) { return act >= ACT_RELU_GLU; }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-// aux: ACT_DECAY's bias of this row
-__device__ __forceinline__ float dense_act(int act, float v, float aux) {
+__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+__device__ __forceinline__ float softcap_f(float z, float cap) { return cap * tanhf(z / cap); }
+// v: the row's product with its bias added; arg: the cap of ACT_SOFTCAP
+__device__ __forceinline__ float dense_act(int act, float v, float arg) {
   switch (act) {
     case ACT_SIGMOID: return sigmoid_f(v);
     case ACT_SILU: return v * sigmoid_f(v);
     case ACT_TANH: return tanhf(v);
-    case ACT_DECAY: return expf(-expf(v + aux));
+    case ACT_DECAY: return expf(-expf(v));
+    case ACT_GELU: return gelu_tanh_f(v);
+    case ACT_SOFTCAP: return softcap_f(v, arg);
     default: return v;
   }
 }
+__device__ __forceinline__ float glu_act(int act, float gate, float up) { return (act == ACT_SILU_GLU ? gate * sigmoid_f(gate) : fmaxf(gate, 0.f)) * up; }
 
 __host__ __device__ __forceinline__ int pad8(int n) { return (n + 7) & ~7; }
 // Gate and up rows of a gated feed-forward share one matrix: eight gate rows, then the same eight up rows.
@@ -42,11 +49,13 @@ constexpr int DGV_WARPS = 16, DGV_THREADS = 32 * DGV_WARPS;
 constexpr int DGV_U = 4;  // 16-byte pieces of each row in flight per lane
 
 struct DgvSeg {
-  const __nv_bfloat16* w;  // [rows][ld] (ACT_RELU_GLU: gate / up rows interleaved, rows = outputs)
+  const __nv_bfloat16* w;  // [rows][ld] (gated products: gate / up rows interleaved, rows = outputs)
   int rows, act;
   float* y;                // [batch][y_stride]
   int y_stride;
   const float* mu;         // token shift: this segment's mix, or nullptr
+  const float* bias;       // [rows], or nullptr
+  float arg;               // cap of ACT_SOFTCAP
 };
 
 struct DgvParams {
@@ -55,7 +64,8 @@ struct DgvParams {
   const float* x;          // [batch][x_stride]
   int x_stride;
   const float* add;        // pending sublayer output [batch][x_stride], or nullptr
-  const float* add_w;      // its norm
+  const float* add_w;      // its norm, or nullptr: added as it is
+  const float* add2;       // further rows added to the stream [batch][x_stride] (only with add), or nullptr
   float* x_out;            // the new residual stream [batch][x_stride] (another buffer than x)
   const float* norm_w;     // nullptr: the input is used as it is
   float eps;
@@ -122,7 +132,7 @@ __global__ void __launch_bounds__(DGV_THREADS, NB <= 2 ? 2 : 1) dense_gemv_kerne
 
   // ---- tasks: pairs of rows ----
   const int seg_fixed = p.ctas_per_seg ? (int)blockIdx.x / p.ctas_per_seg : -1;
-  auto tasks_of = [&](int s) { return p.seg[s].act == ACT_RELU_GLU ? p.seg[s].rows : (p.seg[s].rows + 1) >> 1; };
+  auto tasks_of = [&](int s) { return act_is_glu(p.seg[s].act) ? p.seg[s].rows : (p.seg[s].rows + 1) >> 1; };
   int ntasks = 0, task, stride;
   if (seg_fixed >= 0) {
     ntasks = tasks_of(seg_fixed);
@@ -143,7 +153,7 @@ __global__ void __launch_bounds__(DGV_THREADS, NB <= 2 ? 2 : 1) dense_gemv_kerne
       while (seg + 1 < p.nseg && t >= tasks_of(seg)) { t -= tasks_of(seg); ++seg; }
     }
     const DgvSeg& sg = p.seg[seg];
-    const bool glu = sg.act == ACT_RELU_GLU;
+    const bool glu = act_is_glu(sg.act);
     r0 = glu ? t : 2 * t;
     has1 = glu || r0 + 1 < sg.rows;
     const int64_t a = glu ? glu_row(r0, 0) : r0, b = glu ? glu_row(r0, 1) : (has1 ? r0 + 1 : r0);
@@ -171,7 +181,7 @@ __global__ void __launch_bounds__(DGV_THREADS, NB <= 2 ? 2 : 1) dense_gemv_kerne
   auto slot_of = [&](int n) -> float4* { return reinterpret_cast<float4*>(dgv_x) + (size_t)n * n4; };
   auto place = [&](int j) { return (j & 1) * kc + (j >> 1); };  // float4 j of a vector -> its plane position
   float ss[NB];
-  if (p.add) {
+  if (p.add && p.add_w) {
 #pragma unroll
     for (int n = 0; n < NB; ++n) {
       ss[n] = 0.f;
@@ -193,13 +203,21 @@ __global__ void __launch_bounds__(DGV_THREADS, NB <= 2 ? 2 : 1) dense_gemv_kerne
       continue;
     }
     const size_t row = (size_t)(b0 + n) * p.x_stride;
-    const float f = p.add ? 1.0f / sqrtf(ss[n] / (float)K + p.eps) : 0.f;
+    const float f = p.add && p.add_w ? 1.0f / sqrtf(ss[n] / (float)K + p.eps) : 0.f;
     for (int j = tid; j < n4; j += DGV_THREADS) {
       float4 v = ld4_masked(p.x + row, 4 * j, K);
       if (p.add) {
         const float4 a = ld4_masked(p.add + row, 4 * j, K);
-        const float4 w = ld4_masked(p.add_w, 4 * j, K);
-        v.x += a.x * f * w.x; v.y += a.y * f * w.y; v.z += a.z * f * w.z; v.w += a.w * f * w.w;
+        if (p.add_w) {
+          const float4 w = ld4_masked(p.add_w, 4 * j, K);
+          v.x += a.x * f * w.x; v.y += a.y * f * w.y; v.z += a.z * f * w.z; v.w += a.w * f * w.w;
+        } else {
+          v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+        }
+        if (p.add2) {
+          const float4 e = ld4_masked(p.add2 + row, 4 * j, K);
+          v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+        }
         if (blockIdx.x == 0) *reinterpret_cast<float4*>(p.x_out + row + 4 * j) = v;
       }
       dst[place(j)] = v;
@@ -278,11 +296,11 @@ __global__ void __launch_bounds__(DGV_THREADS, NB <= 2 ? 2 : 1) dense_gemv_kerne
     const int b = b0 + my_col;
     if (my_col < NB && b < p.batch) {
       const DgvSeg& sg = p.seg[seg];
-      if (sg.act == ACT_RELU_GLU) {
-        if (my_row == 0) sg.y[(size_t)b * sg.y_stride + r0] = fmaxf(mine, 0.f) * pair;
+      if (act_is_glu(sg.act)) {
+        if (my_row == 0) sg.y[(size_t)b * sg.y_stride + r0] = glu_act(sg.act, mine, pair);
       } else if (my_row == 0 || has1) {
         const int row = r0 + my_row;
-        float v = dense_act(sg.act, mine, 0.f);
+        float v = dense_act(sg.act, sg.bias ? mine + sg.bias[row] : mine, sg.arg);
         if (p.pen_counts) {
           const int times = p.pen_counts[(size_t)b * p.pen_stride + row];
           const float pen = *p.pen_value;

@@ -23,6 +23,8 @@
 #include "latent_attn.cuh"
 #include "misc.cuh"
 #include "tp.h"
+#include "rglru.cuh"
+#include "shared_kv_attn.cuh"
 #include "wkv.cuh"
 
 namespace b200 {

@@ -5,8 +5,7 @@
 //
 //   latent_append_kernel   prompts: norm + rotation of new rows into the ring, and the rows a chunk attends to laid out
 //                          contiguously (history from the ring, then the new ones) for the key / value expansion
-//   latent_prefill_kernel  prompts: 128 queries of one head per block over expanded keys and values, 64-key tiles, online
-//                          softmax, bfloat16 tensor-core products (mma.sync m16n8k16) with FP32 scores and sums
+//                          that prompt_attn_kernel (attn_tiles.cuh) then runs over
 //   decode                 one token of several sequences: works on the latents themselves. The query's unrotated part is
 //                          taken through W_uk once (q . W_uk c = (W_uk^T q) . c), scores and the weighted sum run over c,
 //                          and the sum is taken through W_uv at the end. latent_decode_kernel does all of it for one
@@ -15,31 +14,9 @@
 //
 // A = type of the cache and of matmul operands: __nv_bfloat16, or float in a 32-bit engine.
 #pragma once
-#include "attn_prefill.cuh"
-#include "block_rows.cuh"
+#include "attn_tiles.cuh"
 
 namespace b200 {
-
-__device__ __forceinline__ float from_operand(float v) { return v; }
-__device__ __forceinline__ float from_operand(__nv_bfloat16 v) { return __bfloat162float(v); }
-// eight consecutive elements (16- or 32-byte aligned)
-__device__ __forceinline__ void load8(const __nv_bfloat16* p, float (&v)[8]) {
-  const uint4 u = *reinterpret_cast<const uint4*>(p);
-  v[0] = bf_lo(u.x); v[1] = bf_hi(u.x); v[2] = bf_lo(u.y); v[3] = bf_hi(u.y);
-  v[4] = bf_lo(u.z); v[5] = bf_hi(u.z); v[6] = bf_lo(u.w); v[7] = bf_hi(u.w);
-}
-__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
-  const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
-  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
-}
-
-// Element i of a rotated vector: pairs (2j, 2j+1) for j < pairs, table row = {cos, sin} per pair; the rest passes.
-__device__ __forceinline__ float rotated(const float* v, int i, const float* rope_row, int pairs) {
-  const int j = i >> 1;
-  if (j >= pairs) return v[i];
-  const float c = rope_row[2 * j], s = rope_row[2 * j + 1];
-  return (i & 1) ? v[i] * c + v[i - 1] * s : v[i] * c - v[i + 1] * s;
-}
 
 struct LatentAppendParams {
   const float* low;    // [T][low_stride]: raw W_dkv h (kv_rank, then rot_dim)
@@ -115,7 +92,8 @@ struct LatentDecodeParams {
   const __nv_bfloat16* uv;  // [heads * vdim][kvp]
   const float* gate;    // [batch][gate_stride]
   int gate_stride;
-  int heads, dim, rot_dim, vdim, kv_rank, window, max_ctx;
+  int heads, dim, rot_dim, vdim, kv_rank, max_ctx;
+  KeyMask mask;
   float scale;
   int nsplit, split_cap;  // context splits per (head, sequence); most keys of one split
   float* part_o;        // [batch][heads][nsplit][kvp]
@@ -199,7 +177,7 @@ __global__ void __launch_bounds__(LAD_THREADS) latent_decode_kernel(const Latent
   }
   A* cache = static_cast<A*>(p.cache) + (size_t)slot * p.cap * p.crow;
   const float* table = p.rope + (size_t)pos * p.pairs * 2;
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, nkeys = pos - lo + 1;
+  const int lo = p.mask.first(pos), nkeys = pos - lo + 1;
   const int chunk = (nkeys + p.nsplit - 1) / p.nsplit;
   const int t0 = lo + split * chunk, t1 = min(pos + 1, t0 + chunk), n = max(0, t1 - t0);
 
@@ -341,27 +319,10 @@ __global__ void __launch_bounds__(LAD_THREADS) latent_decode_kernel(const Latent
   }
 }
 
-__device__ __forceinline__ void lap_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ uint32_t pack_bf2(float a, float b) {
-  const __nv_bfloat162 v = __floats2bfloat162_rn(a, b);
-  return *reinterpret_cast<const uint32_t*>(&v);
-}
-
 // ---- decode on the tensor cores (bfloat16 cache) -------------------------------------------------------------------
 // Three launches: latent_absorb_kernel takes the queries through W_uk and appends the new rows, latent_split_kernel runs
-// scores and weighted sums for 16 heads and one run of keys per block, latent_merge_kernel merges the runs and goes
-// through W_uv. The cached rows are bfloat16 as they are; queries and attention weights enter the products as the sum of
-// two bfloat16 numbers (value and remainder), so that they keep 16 bits of mantissa and the scores FP32 character.
-
-__device__ __forceinline__ void split_bf16(float v, __nv_bfloat16& hi, __nv_bfloat16& lo) {
-  hi = __float2bfloat16(v);
-  lo = __float2bfloat16(v - __bfloat162float(hi));
-}
+// scores and weighted sums for 16 heads and one run of keys per block (split_attend), latent_merge_kernel merges the runs
+// and goes through W_uv.
 
 constexpr int LAB_THREADS = 256;
 constexpr int LAB_COLS = 64;   // latent columns per block
@@ -462,14 +423,6 @@ __global__ void __launch_bounds__(LAB_THREADS) latent_absorb_kernel(const Latent
   }
 }
 
-constexpr int LAS_THREADS = 256, LAS_WARPS = 8, LAS_HEADS = 16, LAS_KEYS = 64;
-
-__host__ __device__ __forceinline__ int las_row(int n) { return (n + 31) / 32 * 32; }
-__host__ __device__ __forceinline__ size_t las_smem_bytes(int crow) {
-  const size_t row = las_row(crow) + 8;
-  return (LAS_KEYS + 2 * LAS_HEADS) * row * 2 + (size_t)2 * LAS_HEADS * (LAS_KEYS + 8) * 2;
-}
-
 struct LatentSplitParams {
   const __nv_bfloat16 *q_hi, *q_lo;  // [batch][heads][qrow]
   int qrow;
@@ -477,7 +430,8 @@ struct LatentSplitParams {
   int crow, kvp, cap;
   const int* positions;
   const int* slots;
-  int heads, window, max_ctx, nsplit;
+  int heads, max_ctx, nsplit;
+  KeyMask mask;
   float* part_o;                     // [batch][heads][nsplit][kvp]
   float* part_ml;                    // [batch][heads][nsplit]{max, sum}, base-e scores
 };
@@ -486,154 +440,53 @@ struct LatentSplitParams {
 template <int TW>
 __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentSplitParams p) {
   extern __shared__ __align__(16) unsigned char las_smem[];
-  __shared__ float mx_s[LAS_WARPS][LAS_HEADS], sum_s[LAS_WARPS][LAS_HEADS];
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  __shared__ SplitStats st;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int split = blockIdx.x, h0 = blockIdx.y * LAS_HEADS, b = blockIdx.z;
-  const int EP = las_row(p.crow), RS = EP + 8, PS = LAS_KEYS + 8;
-  __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(las_smem);
-  __nv_bfloat16* Qh = Ks + LAS_KEYS * RS;
-  __nv_bfloat16* Ql = Qh + LAS_HEADS * RS;
-  __nv_bfloat16* Ph = Ql + LAS_HEADS * RS;
-  __nv_bfloat16* Pl = Ph + LAS_HEADS * PS;
+  const SplitTiles m(las_smem, p.crow);
   pdl_launch_dependents();
   pdl_wait();
   const int pos = p.positions[b];
   if (pos < 0 || pos >= p.max_ctx) return;
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0, nkeys = pos - lo + 1;
+  const int lo = p.mask.first(pos), nkeys = pos - lo + 1;
   const int chunk = ((nkeys + p.nsplit - 1) / p.nsplit + LAS_KEYS - 1) / LAS_KEYS * LAS_KEYS;
   const int k_begin = lo + split * chunk, k_end = min(pos + 1, k_begin + chunk);
   const __nv_bfloat16* cache = p.cache + (size_t)p.slots[b] * p.cap * p.crow;
-  const int nh = min(LAS_HEADS, p.heads - h0), ce = EP >> 3, cc = p.crow >> 3;
+  const int nh = min(LAS_HEADS, p.heads - h0), ce = m.EP >> 3, cc = p.crow >> 3;
   for (int r = warp; r < LAS_HEADS; r += LAS_WARPS) {
     const size_t at = ((size_t)b * p.heads + h0 + min(r, nh - 1)) * p.qrow;
     for (int c = lane; c < ce; c += 32) {
       if (r < nh) {
-        pfa_cp16(Qh + r * RS + 8 * c, p.q_hi + at + 8 * c);
-        pfa_cp16(Ql + r * RS + 8 * c, p.q_lo + at + 8 * c);
+        pfa_cp16(m.Qh + r * m.RS + 8 * c, p.q_hi + at + 8 * c);
+        pfa_cp16(m.Ql + r * m.RS + 8 * c, p.q_lo + at + 8 * c);
       } else {
-        *reinterpret_cast<uint4*>(Qh + r * RS + 8 * c) = make_uint4(0, 0, 0, 0);
-        *reinterpret_cast<uint4*>(Ql + r * RS + 8 * c) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(m.Qh + r * m.RS + 8 * c) = make_uint4(0, 0, 0, 0);
+        *reinterpret_cast<uint4*>(m.Ql + r * m.RS + 8 * c) = make_uint4(0, 0, 0, 0);
       }
     }
   }
   const int tiles = p.kvp >> 3;  // 8-column tiles of the weighted sum; a warp takes pairs of them
   float o[TW][4];
-#pragma unroll
-  for (int i = 0; i < TW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // heads g and g + 8
-  for (int kt = k_begin; kt < k_end; kt += LAS_KEYS) {
-    const int nk = min(LAS_KEYS, k_end - kt);
-    __syncthreads();
-    for (int r = warp; r < LAS_KEYS; r += LAS_WARPS) {
-      const __nv_bfloat16* src = cache + (size_t)((kt + r) % p.cap) * p.crow;
-      __nv_bfloat16* d = Ks + r * RS;
-      for (int c = lane; c < ce; c += 32) {
-        if (r < nk && c < cc) pfa_cp16(d + 8 * c, src + 8 * c);
-        else *reinterpret_cast<uint4*>(d + 8 * c) = make_uint4(0, 0, 0, 0);
-      }
+  auto load_row = [&](int key, __nv_bfloat16* d) {
+    const __nv_bfloat16* src = cache + (size_t)(key % p.cap) * p.crow;
+    for (int c = lane; c < ce; c += 32) {
+      if (c < cc) pfa_cp16(d + 8 * c, src + 8 * c);
+      else *reinterpret_cast<uint4*>(d + 8 * c) = make_uint4(0, 0, 0, 0);
     }
-    pfa_cp_wait_all();
-    __syncthreads();
-    // scores of this warp's 8 keys
-    float s[4] = {0.f, 0.f, 0.f, 0.f}, sl[4] = {0.f, 0.f, 0.f, 0.f};  // products with the queries' values and remainders
-#pragma unroll 2
-    for (int ks = 0; ks < EP; ks += 32) {
-      uint32_t a0[4], a1[4], b0[4], b1[4], kb[4];
-      const int aoff = (lane & 15) * RS + ks + (lane >> 4) * 8;
-      pfa_ldm4(kb, Ks + (warp * 8 + (lane & 7)) * RS + ks + (lane >> 3) * 8);
-      pfa_ldm4(a0, Qh + aoff);
-      pfa_ldm4(a1, Qh + aoff + 16);
-      pfa_ldm4(b0, Ql + aoff);
-      pfa_ldm4(b1, Ql + aoff + 16);
-      lap_mma(s, a0, kb[0], kb[1]);
-      lap_mma(sl, b0, kb[0], kb[1]);
-      lap_mma(s, a1, kb[2], kb[3]);
-      lap_mma(sl, b1, kb[2], kb[3]);
-    }
-    float x0 = -INFINITY, x1 = -INFINITY;
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const bool ok = warp * 8 + 2 * t + e < nk;
-      s[e] = ok ? s[e] + sl[e] : -INFINITY;
-      s[2 + e] = ok ? s[2 + e] + sl[2 + e] : -INFINITY;
-      x0 = fmaxf(x0, s[e]);
-      x1 = fmaxf(x1, s[2 + e]);
-    }
-#pragma unroll
-    for (int x = 1; x < 4; x <<= 1) {
-      x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, x));
-      x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, x));
-    }
-    if (t == 0) { mx_s[warp][g] = x0; mx_s[warp][g + 8] = x1; }
-    __syncthreads();
-    float n0 = m0, n1 = m1;
-#pragma unroll
-    for (int w = 0; w < LAS_WARPS; ++w) {
-      n0 = fmaxf(n0, mx_s[w][g]);
-      n1 = fmaxf(n1, mx_s[w][g + 8]);
-    }
-    const float f0 = expf(m0 - n0), f1 = expf(m1 - n1);  // every tile has a key, so n is finite
-    m0 = n0; m1 = n1;
-    float y0 = 0.f, y1 = 0.f;
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int k = warp * 8 + 2 * t + e;
-      const float w0 = expf(s[e] - n0), w1 = expf(s[2 + e] - n1);
-      y0 += w0; y1 += w1;
-      split_bf16(w0, Ph[g * PS + k], Pl[g * PS + k]);
-      split_bf16(w1, Ph[(g + 8) * PS + k], Pl[(g + 8) * PS + k]);
-    }
-    l0 = l0 * f0 + y0; l1 = l1 * f1 + y1;  // this thread's share; shares of lanes and warps are added at the end
-#pragma unroll
-    for (int i = 0; i < TW; ++i) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
-    __syncthreads();
-    // weighted sums: this warp's pairs of column tiles
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-      uint32_t ah[4], al[4];
-      const int aoff = (lane & 15) * PS + kk * 16 + (lane >> 4) * 8;
-      pfa_ldm4(ah, Ph + aoff);
-      pfa_ldm4(al, Pl + aoff);
-#pragma unroll
-      for (int i = 0; i < TW / 2; ++i) {
-        const int tile = 2 * (warp + LAS_WARPS * i);
-        if (tile < tiles) {  // an odd last tile reads the row's next eight columns and drops them
-          uint32_t vb[4];
-          pfa_ldm4t(vb, Ks + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * RS + tile * 8 + (lane >> 4) * 8);
-          lap_mma(o[2 * i], ah, vb[0], vb[1]);
-          lap_mma(o[2 * i + 1], ah, vb[2], vb[3]);
-          lap_mma(o[2 * i], al, vb[0], vb[1]);
-          lap_mma(o[2 * i + 1], al, vb[2], vb[3]);
-        }
-      }
-    }
-  }
-#pragma unroll
-  for (int x = 1; x < 4; x <<= 1) {
-    l0 += __shfl_xor_sync(0xffffffffu, l0, x);
-    l1 += __shfl_xor_sync(0xffffffffu, l1, x);
-  }
-  __syncthreads();
-  if (t == 0) { sum_s[warp][g] = l0; sum_s[warp][g + 8] = l1; mx_s[warp][g] = m0; mx_s[warp][g + 8] = m1; }
-  __syncthreads();
+  };
+  split_attend<TW>(m, st, k_begin, k_end, 0, tiles, load_row, [](float s) { return s; }, o);
   const size_t row = ((size_t)b * p.heads + h0) * p.nsplit + split;
   if (tid < nh) {
     float* ml = p.part_ml + (row + (size_t)tid * p.nsplit) * 2;
-    ml[0] = mx_s[0][tid];
+    ml[0] = st.mx[0][tid];
     float l = 0.f;
-    for (int w = 0; w < LAS_WARPS; ++w) l += sum_s[w][tid];
+    for (int w = 0; w < LAS_WARPS; ++w) l += st.sum[w][tid];
     ml[1] = k_begin < k_end ? l : 0.f;
   }
   if (k_begin >= k_end) return;  // an empty run: its sum of zero makes the merge skip it
-#pragma unroll
-  for (int i = 0; i < TW; ++i) {
-    const int tile = 2 * (warp + LAS_WARPS * (i >> 1)) + (i & 1);
-    if (tile < tiles) {
-      const int c = 8 * tile + 2 * t;
-      if (g < nh) *reinterpret_cast<float2*>(p.part_o + (row + (size_t)g * p.nsplit) * p.kvp + c) = make_float2(o[i][0], o[i][1]);
-      if (g + 8 < nh) *reinterpret_cast<float2*>(p.part_o + (row + (size_t)(g + 8) * p.nsplit) * p.kvp + c) = make_float2(o[i][2], o[i][3]);
-    }
-  }
+  split_columns<TW>(o, tiles, nh, [&](int h, int c, float x, float y) {
+    *reinterpret_cast<float2*>(p.part_o + (row + (size_t)h * p.nsplit) * p.kvp + c) = make_float2(x, y);
+  });
 }
 
 constexpr int LAM_THREADS = 256, LAM_ROWS = 32;  // value rows per block: four per warp
@@ -714,238 +567,6 @@ __global__ void __launch_bounds__(LAM_THREADS) latent_merge_kernel(const LatentD
     const float v = lane == 0 ? acc[0] : lane == 1 ? acc[1] : lane == 2 ? acc[2] : acc[3];
     const int j = h * p.vdim + r0 + lane;
     static_cast<O*>(p.out)[(size_t)b * p.out_stride + j] = to_operand<O>(v * p.gate[(size_t)b * p.gate_stride + j]);
-  }
-}
-
-// ---- prompts -----------------------------------------------------------------------------------------------------
-constexpr int LAP_Q = 128, LAP_K = 64, LAP_THREADS = 256, LAP_WARPS = 8;
-
-struct LatentPrefillParams {
-  const float* q;            // [T][q_stride], unrotated
-  int q_stride;
-  const float* rope;
-  int pairs;
-  const __nv_bfloat16* kv;   // [context rows][kv_stride]: unrotated keys of all heads, values from column v_off on
-  int kv_stride, v_off;
-  const __nv_bfloat16* kr;   // [context rows][kr_stride] rotated key parts
-  int kr_stride;
-  const float* gate;         // [T][gate_stride]
-  int gate_stride;
-  const RunDesc* runs;
-  int heads, dim, rot_dim, vdim, window;
-  float scale;
-  __nv_bfloat16* out;        // [T][out_stride]
-  int out_stride;
-};
-
-__host__ __device__ __forceinline__ int lap_qk_stride(int dim, int rot) { return (dim + rot + 15) / 16 * 16 + 8; }
-__host__ __device__ __forceinline__ int lap_value_cols(int vdim) { return vdim <= 32 ? 32 : vdim <= 64 ? 64 : vdim <= 128 ? 128 : 256; }
-__host__ __device__ __forceinline__ size_t lap_smem_bytes(int dim, int rot, int vp) {
-  return ((size_t)(LAP_Q + LAP_K) * lap_qk_stride(dim, rot) + (size_t)LAP_K * (vp + 8)) * 2;
-}
-
-// grid = (query blocks of the longest run, heads, runs). VP = value columns per head rounded up to 32, 64, 128 or 256.
-template <int VP>
-__global__ void __launch_bounds__(LAP_THREADS, VP <= 128 ? 2 : 1) latent_prefill_kernel(const LatentPrefillParams p) {
-  extern __shared__ __align__(16) unsigned char lap_smem[];
-  const RunDesc run = p.runs[blockIdx.z];
-  const int q0 = blockIdx.x * LAP_Q, h = blockIdx.y;
-  if (q0 >= run.len) return;
-  const int E = p.dim + p.rot_dim, EP = (E + 15) / 16 * 16, QS = EP + 8;
-  constexpr int VS = VP + 8, NT_O = VP / 8;
-  __nv_bfloat16* Qs = reinterpret_cast<__nv_bfloat16*>(lap_smem);
-  __nv_bfloat16* Ks = Qs + LAP_Q * QS;
-  __nv_bfloat16* Vs = Ks + LAP_K * QS;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
-  const int nq = min(LAP_Q, run.len - q0);
-  const bool vec = !((p.dim | p.rot_dim | p.vdim | p.kv_stride | p.v_off | p.kr_stride | p.q_stride) & 7);
-  // queries, rotated; the scale is applied to the products
-  if (vec) {  // pieces of four elements (two pairs), eight of them in flight per thread
-    const int n4 = EP >> 2, d4 = p.dim >> 2, e4 = E >> 2;
-    for (int i0 = tid; i0 < LAP_Q * n4; i0 += 8 * LAP_THREADS) {
-      float4 v[8], cs[8];
-#pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const int i = i0 + k * LAP_THREADS, r = i / n4, c = i - r * n4;
-        const bool ok = r < nq && c < e4;
-        v[k] = ok ? *reinterpret_cast<const float4*>(p.q + (size_t)(run.row0 + q0 + r) * p.q_stride + h * E + 4 * c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        cs[k] = make_float4(1.f, 0.f, 1.f, 0.f);  // pairs beyond the rotated ones pass
-        const int j = 2 * (c - d4);               // first of the piece's two pairs
-        if (ok && j >= 0) {
-          const float* table = p.rope + ((size_t)(run.start + q0 + r) * p.pairs + j) * 2;
-          if (j < p.pairs) { cs[k].x = table[0]; cs[k].y = table[1]; }
-          if (j + 1 < p.pairs) { cs[k].z = table[2]; cs[k].w = table[3]; }
-        }
-      }
-#pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const int i = i0 + k * LAP_THREADS, r = i / n4, c = i - r * n4;
-        if (r < LAP_Q)
-          *reinterpret_cast<uint2*>(Qs + r * QS + 4 * c) = make_uint2(pack_bf2(v[k].x * cs[k].x - v[k].y * cs[k].y, v[k].y * cs[k].x + v[k].x * cs[k].y),
-                                                                      pack_bf2(v[k].z * cs[k].z - v[k].w * cs[k].w, v[k].w * cs[k].z + v[k].z * cs[k].w));
-      }
-    }
-  } else {
-    for (int r = warp; r < LAP_Q; r += LAP_WARPS) {
-      const float* qr = p.q + (size_t)(run.row0 + q0 + min(r, nq - 1)) * p.q_stride + h * E;
-      const float* table = p.rope + (size_t)(run.start + q0 + min(r, nq - 1)) * p.pairs * 2;
-      for (int c = lane; c < EP; c += 32) {
-        float v = 0.f;
-        if (r < nq && c < E) v = c < p.dim ? qr[c] : rotated(qr + p.dim, c - p.dim, table, p.pairs);
-        Qs[r * QS + c] = __float2bfloat16(v);
-      }
-    }
-  }
-  const int qpos0 = run.start + q0;                       // position of the block's first query
-  const int kfirst = p.window > 0 ? max(0, qpos0 - p.window + 1) : 0, klast = qpos0 + nq - 1;
-  const int base = run.start - run.hist;                  // position of the run's first context row
-  const int my0 = qpos0 + warp * 16 + g, my1 = my0 + 8;   // this thread's two query positions
-  const int win = p.window > 0 ? p.window : 0x7fffffff;
-  float o[NT_O][4];
-#pragma unroll
-  for (int i = 0; i < NT_O; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-  const float sc2 = p.scale * 1.4426950408889634f;
-
-  // Key and value tiles have one buffer each: the next key tile is requested as soon as this one's scores are done, the
-  // next value tile after this one's products, so each copy runs under the other half of the work.
-  auto load_k = [&](int kt) {
-    const int nk = min(LAP_K, klast - kt + 1);
-    const size_t crow = (size_t)(run.ctx0 + kt - base);
-    if (vec) {
-      const int ce = EP >> 3, cd = p.dim >> 3, cn = E >> 3;
-      for (int r = warp; r < LAP_K; r += LAP_WARPS) {
-        const __nv_bfloat16* kv = p.kv + (crow + r) * p.kv_stride + h * p.dim;
-        const __nv_bfloat16* kr = p.kr + (crow + r) * p.kr_stride;
-        for (int c = lane; c < ce; c += 32) {
-          __nv_bfloat16* d = Ks + r * QS + 8 * c;
-          if (r < nk && c < cn) pfa_cp16(d, c < cd ? kv + 8 * c : kr + 8 * (c - cd));
-          else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
-        }
-      }
-    } else {
-      for (int i = tid; i < LAP_K * EP; i += LAP_THREADS) {
-        const int r = i / EP, c = i - r * EP;
-        __nv_bfloat16 v = __float2bfloat16(0.f);
-        if (r < nk && c < E) v = c < p.dim ? p.kv[(crow + r) * p.kv_stride + h * p.dim + c] : p.kr[(crow + r) * p.kr_stride + c - p.dim];
-        Ks[r * QS + c] = v;
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  auto load_v = [&](int kt) {
-    const int nk = min(LAP_K, klast - kt + 1);
-    const size_t crow = (size_t)(run.ctx0 + kt - base);
-    if (vec) {
-      constexpr int CV = VP >> 3;
-      const int cvn = p.vdim >> 3;
-      for (int i = tid; i < LAP_K * CV; i += LAP_THREADS) {
-        const int r = i / CV, c = i % CV;
-        __nv_bfloat16* d = Vs + r * VS + 8 * c;
-        if (r < nk && c < cvn) pfa_cp16(d, p.kv + (crow + r) * p.kv_stride + p.v_off + h * p.vdim + 8 * c);
-        else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
-      }
-    } else {
-      for (int i = tid; i < LAP_K * VP; i += LAP_THREADS) {
-        const int r = i / VP, c = i - r * VP;
-        Vs[r * VS + c] = r < nk && c < p.vdim ? p.kv[(crow + r) * p.kv_stride + p.v_off + h * p.vdim + c] : __float2bfloat16(0.f);
-      }
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  load_k(kfirst);
-  load_v(kfirst);
-  for (int kt = kfirst; kt <= klast; kt += LAP_K) {
-    asm volatile("cp.async.wait_group 1;" ::: "memory");  // the key tile; its value tile may still be on its way
-    __syncthreads();
-    // scores: 16 queries x 64 keys per warp
-    float s[8][4];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-    for (int ks = 0; ks < EP; ks += 16) {
-      uint32_t a[4];
-      pfa_ldm4(a, Qs + (warp * 16 + (lane & 15)) * QS + ks + (lane >> 4) * 8);
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {  // 16 keys: two 8-key fragments
-        uint32_t kb[4];
-        pfa_ldm4(kb, Ks + (nt * 16 + (lane & 7) + (lane >> 4) * 8) * QS + ks + ((lane >> 3) & 1) * 8);
-        lap_mma(s[2 * nt], a, kb[0], kb[1]);
-        lap_mma(s[2 * nt + 1], a, kb[2], kb[3]);
-      }
-    }
-    __syncthreads();  // every warp has read the key tile
-    if (kt + LAP_K <= klast) load_k(kt + LAP_K);
-    else asm volatile("cp.async.commit_group;" ::: "memory");  // keeps one group per step
-    float n0 = m0, n1 = m1;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int key = kt + 8 * i + 2 * t + e;
-        s[i][e] = key <= my0 && my0 - key < win ? s[i][e] * sc2 : -INFINITY;
-        s[i][2 + e] = key <= my1 && my1 - key < win ? s[i][2 + e] * sc2 : -INFINITY;
-        n0 = fmaxf(n0, s[i][e]);
-        n1 = fmaxf(n1, s[i][2 + e]);
-      }
-    }
-#pragma unroll
-    for (int x = 1; x < 4; x <<= 1) {
-      n0 = fmaxf(n0, __shfl_xor_sync(0xffffffffu, n0, x));
-      n1 = fmaxf(n1, __shfl_xor_sync(0xffffffffu, n1, x));
-    }
-    // a row that has seen no key yet keeps -infinity: subtract 0 then, every weight is exp2(-inf) = 0
-    const float z0 = n0 == -INFINITY ? 0.f : n0, z1 = n1 == -INFINITY ? 0.f : n1;
-    const float f0 = exp2f(m0 - z0), f1 = exp2f(m1 - z1);
-    m0 = n0; m1 = n1;
-    l0 *= f0; l1 *= f1;
-#pragma unroll
-    for (int i = 0; i < NT_O; ++i) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        s[i][e] = exp2f(s[i][e] - z0);
-        s[i][2 + e] = exp2f(s[i][2 + e] - z1);
-        l0 += s[i][e];
-        l1 += s[i][2 + e];
-      }
-    }
-    asm volatile("cp.async.wait_group 1;" ::: "memory");  // the value tile
-    __syncthreads();
-    // weighted values
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-      const uint32_t a[4] = {pack_bf2(s[2 * kk][0], s[2 * kk][1]), pack_bf2(s[2 * kk][2], s[2 * kk][3]), pack_bf2(s[2 * kk + 1][0], s[2 * kk + 1][1]),
-                             pack_bf2(s[2 * kk + 1][2], s[2 * kk + 1][3])};
-#pragma unroll
-      for (int nt = 0; nt < NT_O / 2; ++nt) {
-        uint32_t vb[4];
-        pfa_ldm4t(vb, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + nt * 16 + (lane >> 4) * 8);
-        lap_mma(o[2 * nt], a, vb[0], vb[1]);
-        lap_mma(o[2 * nt + 1], a, vb[2], vb[3]);
-      }
-    }
-    __syncthreads();  // every warp has read the value tile
-    if (kt + LAP_K <= klast) load_v(kt + LAP_K);
-    else asm volatile("cp.async.commit_group;" ::: "memory");
-  }
-#pragma unroll
-  for (int x = 1; x < 4; x <<= 1) {
-    l0 += __shfl_xor_sync(0xffffffffu, l0, x);
-    l1 += __shfl_xor_sync(0xffffffffu, l1, x);
-  }
-  const float i0 = 1.0f / l0, i1 = 1.0f / l1;
-#pragma unroll
-  for (int i = 0; i < NT_O; ++i) {
-#pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int r = warp * 16 + g + (e >> 1) * 8, c = 8 * i + 2 * t + (e & 1);
-      if (r < nq && c < p.vdim) {
-        const size_t row = (size_t)(run.row0 + q0 + r);
-        const int j = h * p.vdim + c;
-        p.out[row * p.out_stride + j] = __float2bfloat16(o[i][e] * (e < 2 ? i0 : i1) * p.gate[row * p.gate_stride + j]);
-      }
-    }
   }
 }
 

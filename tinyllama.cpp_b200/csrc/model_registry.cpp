@@ -37,6 +37,11 @@ std::vector<int> BlockSpec::runs() const {
   return out;
 }
 
+bool BlockSpec::begins_further_pass(int run) const {
+  const int n = loop_stop - loop_start, at = run - loop_start;
+  return n > 0 && at > 0 && at < n * loop_times && at % n == 0;
+}
+
 std::vector<TensorNeed> block_tensor_needs(const BlockSpec& s) {
   std::vector<TensorNeed> out;
   const int64_t W = s.width;
@@ -46,7 +51,7 @@ std::vector<TensorNeed> block_tensor_needs(const BlockSpec& s) {
     const MixerSpec& m = y.mix;
     const std::string L = "l" + std::to_string(l) + ".";
     out.push_back({L + "norm1", {W}});
-    out.push_back({L + "norm1b", {W}});
+    if (s.post_norm) out.push_back({L + "norm1b", {W}});
     const int64_t H = m.heads, D = m.dim;
     if (m.kind == MixerKind::LatentAttention) {
       out.push_back({L + "mix.dq", {m.q_rank, W}});
@@ -58,6 +63,24 @@ std::vector<TensorNeed> block_tensor_needs(const BlockSpec& s) {
       out.push_back({L + "mix.uv", {H * m.vdim, m.kv_rank}});
       out.push_back({L + "mix.g", {H * m.vdim, W}});
       out.push_back({L + "mix.o", {W, H * m.vdim}});
+    } else if (m.kind == MixerKind::SharedKvAttention) {
+      out.push_back({L + "mix.q", {H * D, W}});
+      out.push_back({L + "mix.k", {m.kv_heads * D, W}});
+      out.push_back({L + "mix.o", {W, H * D}});
+    } else if (m.kind == MixerKind::RgLru) {
+      const int64_t N = m.width, B = m.blocks, S = N / B;
+      for (const char* k : {"y", "x"}) {
+        out.push_back({L + "mix." + k, {N, W}});
+        out.push_back({L + "mix." + k + ".b", {N}});
+      }
+      out.push_back({L + "mix.conv", {N, m.conv}});
+      out.push_back({L + "mix.conv.b", {N}});
+      for (const char* k : {"ra", "ri"}) {
+        out.push_back({L + "mix." + k, {B, S, S}});
+        out.push_back({L + "mix." + k + ".b", {B, S}});
+      }
+      out.push_back({L + "mix.lam", {N}});
+      out.push_back({L + "mix.o", {W, N}});
     } else {
       for (const char* k : {"r", "k", "v", "g", "w"}) out.push_back({L + "mix.mu." + k, {W}});
       for (const char* k : {"r", "k", "v", "g"}) out.push_back({L + "mix." + k, {H * D, W}});
@@ -70,14 +93,14 @@ std::vector<TensorNeed> block_tensor_needs(const BlockSpec& s) {
     }
     if (y.ff) {
       out.push_back({L + "norm2", {W}});
-      out.push_back({L + "norm2b", {W}});
+      if (s.post_norm) out.push_back({L + "norm2b", {W}});
       out.push_back({L + "mlp.gate", {y.ff, W}});
       out.push_back({L + "mlp.up", {y.ff, W}});
       out.push_back({L + "mlp.down", {W, y.ff}});
     }
   }
   out.push_back({"final.norm", {W}});
-  out.push_back({"head", {s.vocab, W}});
+  if (!s.tied_head) out.push_back({"head", {s.vocab, W}});
   return out;
 }
 
@@ -115,40 +138,59 @@ static MixerSpec read_latent_attention(const Json& j) {
   if (const Json* r = j.find("rot")) m.rot = read_rot(*r);
   if (m.rot.dims > m.rot_dim) throw std::runtime_error("rot.dims exceeds rot_dim");
   if (const Json* k = j.find("mask"))
-    if (k->find("size")) m.window = positive(*k, "size");
+    if (k->find("size")) m.mask.size = positive(*k, "size");
   return m;
 }
 
-static BlockSpec read_nezolix(const Json& c, const StFile& weights) {
+static MixerSpec read_shared_kv_attention(const Json& j) {
+  MixerSpec m;
+  m.kind = MixerKind::SharedKvAttention;
+  m.heads = positive(j, "heads");
+  m.kv_heads = positive(j, "kv_heads");
+  m.dim = m.vdim = positive(j, "dim");
+  m.sink = true;
+  m.scale = j.number("scale");
+  if (j.find("softcap")) m.softcap = j.number("softcap");
+  if (m.heads % m.kv_heads) throw std::runtime_error("heads must be a multiple of kv_heads");
+  if (j.find("vdim") && j.integer("vdim") != m.dim) throw std::runtime_error("vdim must equal dim: the values are the keys");
+  if (m.softcap < 0) throw std::runtime_error("softcap must be positive");
+  if (const Json* r = j.find("rot")) m.rot = read_rot(*r);
+  if (m.rot.dims > m.dim) throw std::runtime_error("rot.dims exceeds dim");
+  if (const Json* k = j.find("mask"))
+    if (k->find("size")) m.mask = {positive(*k, "size"), true};
+  return m;
+}
+
+static MixerSpec read_rglru(const Json& j) {
+  MixerSpec m;
+  m.kind = MixerKind::RgLru;
+  m.width = positive(j, "width");
+  m.blocks = positive(j, "blocks");
+  m.conv = positive(j, "conv");
+  if (m.width % m.blocks) throw std::runtime_error("width must be a multiple of blocks");
+  return m;
+}
+
+// What the block architectures' config.json files share: sizes, the layer list (mixer: type, entry, layer index -> its
+// description) and the loop.
+template <typename Mixer>
+static BlockSpec read_stack(const Json& c, GluKind glu, Mixer mixer) {
   BlockSpec s;
   s.arch = c.text("architecture");
   s.vocab = positive(c, "vocab");
   s.width = positive(c, "width");
   s.eps = c.at("norm").number("eps");
-  if (const Json* e = c.find("embedding"))
-    if (e->find("scale")) s.embed_scale = e->number("scale");
   const Json& layers = c.at("layers");
   if (layers.kind != Json::Array || layers.items.empty()) throw std::runtime_error("'layers' must be a non-empty list");
   for (size_t l = 0; l < layers.items.size(); ++l) {
     const Json& e = layers.items[l];
-    const std::string& type = e.text("type");
+    const std::string where = "layer " + std::to_string(l) + ": ";
     LayerSpec y;
-    if (type == "latent_attention") {
-      y.mix = read_latent_attention(e.at("mixer"));
-    } else if (type == "wkv") {
-      y.mix.kind = MixerKind::Wkv;
-      y.mix.heads = positive(e.at("mixer"), "heads");
-      y.mix.dim = positive(e.at("mixer"), "dim");
-      const auto it = weights.tensors.find("l" + std::to_string(l) + ".mix.w1");
-      if (it == weights.tensors.end() || it->second.shape.size() != 2 || it->second.shape[0] < 1)
-        throw std::runtime_error("layer " + std::to_string(l) + ": decay matrix w1 is missing");
-      y.mix.decay_rank = (int)it->second.shape[0];
-    } else {
-      throw std::runtime_error("layer " + std::to_string(l) + ": unknown mixer '" + type + "'");
-    }
+    if (!mixer(e.text("type"), e.at("mixer"), l, y.mix)) throw std::runtime_error(where + "unknown mixer '" + e.text("type") + "'");
     if (const Json* f = e.find("mlp")) {
-      if (f->text("kind") != "dense") throw std::runtime_error("layer " + std::to_string(l) + ": unknown feed-forward '" + f->text("kind") + "'");
+      if (f->text("kind") != "dense") throw std::runtime_error(where + "unknown feed-forward '" + f->text("kind") + "'");
       y.ff = positive(*f, "ff");
+      y.glu = glu;
     }
     s.layers.push_back(y);
   }
@@ -162,9 +204,48 @@ static BlockSpec read_nezolix(const Json& c, const StFile& weights) {
   return s;
 }
 
+static BlockSpec read_nezolix(const Json& c, const StFile& weights) {
+  BlockSpec s = read_stack(c, GluKind::Relu, [&](const std::string& type, const Json& j, size_t l, MixerSpec& m) {
+    if (type == "latent_attention") {
+      m = read_latent_attention(j);
+    } else if (type == "wkv") {
+      m.kind = MixerKind::Wkv;
+      m.heads = positive(j, "heads");
+      m.dim = positive(j, "dim");
+      const auto it = weights.tensors.find("l" + std::to_string(l) + ".mix.w1");
+      if (it == weights.tensors.end() || it->second.shape.size() != 2 || it->second.shape[0] < 1)
+        throw std::runtime_error("layer " + std::to_string(l) + ": decay matrix w1 is missing");
+      m.decay_rank = (int)it->second.shape[0];
+    } else {
+      return false;
+    }
+    return true;
+  });
+  if (const Json* e = c.find("embedding"))
+    if (e->find("scale")) s.embed_scale = e->number("scale");
+  return s;
+}
+
+static BlockSpec read_pizilix(const Json& c, const StFile&) {
+  BlockSpec s = read_stack(c, GluKind::Silu, [](const std::string& type, const Json& j, size_t, MixerSpec& m) {
+    if (type == "attention") m = read_shared_kv_attention(j);
+    else if (type == "rglru") m = read_rglru(j);
+    else return false;
+    return true;
+  });
+  s.post_norm = false;
+  s.norm_offset = 1.0;
+  s.tied_head = true;
+  s.loop_adds_embedding = true;
+  if (c.find("logit_softcap")) s.logit_softcap = c.number("logit_softcap");
+  if (s.logit_softcap < 0) throw std::runtime_error("logit_softcap must be positive");
+  return s;
+}
+
 static const ArchEntry ARCHS[] = {
     {"llama", true, nullptr},
     {"Nezolix", false, read_nezolix},
+    {"Pizilix", false, read_pizilix},
 };
 
 const ArchEntry* find_arch(const std::string& name) {
