@@ -8,11 +8,11 @@ the Llama-2-7B-shaped Q4_K_M-style model at batch 1 with a 1024-token prompt and
 Weights are synthetic (seeded N(0, 0.02), quantized by the package's writer); prompts are seeded
 uniform token ids. One JSON line is printed by rank 0.
 
-  python bench.py --block-model nezolix-w4096 [--steps K] [--warmup W]
+  python bench.py --block-model nezolix-w4096|nezolix-w2048|pizilix-w4096|pizilix-w2048 [--steps K] [--warmup W]
 
 measures a block model instead (random bfloat16 weights in the sizes of a real model's layers): prompt ingestion and
-decode throughput, and every kind of launch alone, beside a packed-weight Llama model of the same width, feed-forward
-size, heads, layers and vocabulary.
+decode throughput, and every kind of launch alone, beside the closest other model of the same width, feed-forward size,
+heads, layers and vocabulary: for Nezolix a packed-weight Llama model, for Pizilix Nezolix.
 """
 import argparse
 import json
@@ -239,9 +239,16 @@ def parity_in_run(eng, shape, scheme, kv):
 def block_kinds(shape, batch, rows, chunk, context):
     """FLOPs of each timed kind of a block model's launch (selector -> name, FLOPs per launch)."""
     s = shape
-    H, D, R, V, W = s["heads"], s["dim"], s["rot_dim"], s["vdim"], s["width"]
     T = chunk if rows else batch
     win = min(s["window"], context)
+    if s["design"] == "Pizilix":
+        H, G, D, W, N, bs = s["heads"], s["kv_heads"], s["dim"], s["width"], s["lru_width"], s["lru_width"] // s["lru_blocks"]
+        keys = (win + 1) / 2 if rows else win  # a chunk of the timed length starts at a border of the mask's chunks
+        kinds = {0: ("gate_up", 2 * 2 * s["ff"] * W * T), 2: ("o_proj", 2 * W * H * D * T), 3: ("down_proj", 2 * W * s["ff"] * T), 32: ("attention_in (q, k)", 2 * (H + G) * D * W * T),
+                 33: ("attention", int(2 * H * T * keys * 2 * D)), 35: ("lru_in (y, x)", 2 * 2 * N * W * T), 36: ("lru_gates_recurrence", 2 * 2 * N * bs * T)}
+        kinds.update({34: ("attention_append", 0), 37: ("lru_apply", 0), 11: ("norm_rows", 0)} if rows else {4: ("lm_head", 2 * s["vocab"] * W * T)})
+        return kinds
+    H, D, R, V, W = s["heads"], s["dim"], s["rot_dim"], s["vdim"], s["width"]
     ctx = min(s["window"] - 1, context - chunk) + chunk
     hd = s["wkv_heads"] * s["wkv_dim"]
     kinds = {0: ("gate_up", 2 * 2 * s["ff"] * W * T), 1: ("latent_in (W_dq, W_dkv, gate)", 2 * (s["q_rank"] + s["kv_rank"] + R + H * V) * W * T),
@@ -256,20 +263,27 @@ def block_kinds(shape, batch, rows, chunk, context):
 
 
 def run_block(args):
-    """Prompt and decode throughput of a block model and of the packed-weight model of equal size, one JSON line."""
+    """Prompt and decode throughput of a block model and of the closest model of equal size, one JSON line."""
     pkg = __graft_entry__.load_package()
     json_fd = os.dup(1)
     os.dup2(2, 1)
     shape = pkg.synth.BLOCK_SHAPES[args.block_model]
     base = "/dev/shm" if os.path.isdir("/dev/shm") and os.access("/dev/shm", os.W_OK) else "/tmp"
-    folder = os.path.join(base, f"b200_synth_{args.block_model}")
-    if not os.path.exists(os.path.join(folder, "done")):
-        pkg.synth.write_block_model(folder, args.block_model)
-        open(os.path.join(folder, "done"), "w").close()
-    like = dict(hidden=shape["width"], ffn=shape["ff"], n_heads=shape["heads"], n_kv_heads=shape["heads"], n_layers=shape["n_layers"], vocab=shape["vocab"],
+
+    def block_folder(name):
+        folder = os.path.join(base, f"b200_synth_{name}")
+        if not os.path.exists(os.path.join(folder, "done")):
+            pkg.synth.write_block_model(folder, name)
+            open(os.path.join(folder, "done"), "w").close()
+        return folder
+
+    folder = block_folder(args.block_model)
+    like_name = args.block_model.replace("pizilix", "nezolix") if shape["design"] == "Pizilix" else None  # None: the packed model
+    like = pkg.synth.BLOCK_SHAPES[like_name] if like_name else dict(hidden=shape["width"], ffn=shape["ff"], n_heads=shape["heads"], n_kv_heads=shape["heads"], n_layers=shape["n_layers"], vocab=shape["vocab"],
                 max_pos=8192, theta=10000.0)
     gguf = os.path.join(base, f"b200_synth_like_{args.block_model}.gguf")
-    if not os.path.exists(gguf):
+    like_folder = block_folder(like_name) if like_name else None
+    if not like_name and not os.path.exists(gguf):
         pkg.synth.write_gguf(gguf + ".tmp", like, scheme=0)
         os.replace(gguf + ".tmp", gguf)
     progress("model files ready")
@@ -323,23 +337,34 @@ def run_block(args):
         return {"us": round(us, 2), "bytes": int(nbytes), "GFLOP": round(flops / 1e9, 3), "bound": "hbm" if t_mem >= t_math else "math",
                 "frac": round(max(t_mem, t_math) / us, 4)}
 
-    def block(b, ctx):
-        return pkg.Engine.from_model(folder, max_seqs=b, max_ctx=ctx)
+    def block(b, ctx, path=folder):
+        return pkg.Engine.from_model(path, max_seqs=b, max_ctx=ctx)
 
     def packed(b, ctx):
         return pkg.Engine.from_gguf(gguf, kv_dtype=pkg.KV_I8, max_seqs=b, max_ctx=ctx)
 
-    result = {"block model": throughput(block, "bf16, bf16 latent cache, window %d" % shape["window"]), "packed model": throughput(packed, "Q8_0, INT8 KV cache")}
+    note = "bf16, bf16 cache, window %d" % shape["window"]
+    result = {"block model": throughput(block, note)}
+    if like_name:
+        result[like_name] = throughput(lambda b, ctx: block(b, ctx, like_folder), note)
+    else:
+        result["packed model"] = throughput(packed, "Q8_0, INT8 KV cache")
     progress("throughput done")
     kernels = {}
-    for label, b, rows in (("decode batch 1", 1, False), ("decode batch 4", 4, False), (f"prompt chunk of {chunk}", 1, True)):
-        eng = block(b, 4096)
-        kernels[label] = {}
-        for which, (name, flops) in block_kinds(shape, b, rows, chunk, 4096).items():
-            us, nbytes = eng.time_kernel(which + (16 if rows else 0), 48)
-            kernels[label][name] = frac(us, nbytes, flops, fp32=which == 8 or (which == 6 and not rows))
-        eng.close()
-    for label, b, rows in (("packed: decode batch 1", 1, False), ("packed: prompt chunk of 512", 512, True)):
+
+    def time_block(name, path, shp):
+        for label, b, rows in (("decode batch 1", 1, False), ("decode batch 4", 4, False), (f"prompt chunk of {chunk}", 1, True)):
+            eng = block(b, 4096, path)
+            out = kernels[name + label] = {}
+            for which, (kind, flops) in block_kinds(shp, b, rows, chunk, 4096).items():
+                us, nbytes = eng.time_kernel(which + (16 if rows else 0), 48)
+                out[kind] = frac(us, nbytes, flops, fp32=not rows and which in (6, 33, 36) or which == 8)
+            eng.close()
+
+    time_block("", folder, shape)
+    if like_name:
+        time_block(like_name + ": ", like_folder, like)
+    for label, b, rows in () if like_name else (("packed: decode batch 1", 1, False), ("packed: prompt chunk of 512", 512, True)):
         eng = packed(b, 4096 if b == 1 else 16)
         names = {0: "gate_up", 1: "qkv", 2: "o_proj", 3: "down_proj"}
         T, W, F = (512 if rows else 1), like["hidden"], like["ffn"]
@@ -349,16 +374,17 @@ def run_block(args):
             us, nbytes = eng.time_kernel(which + (16 if rows else 0), 48)
             kernels[label][name] = frac(us, nbytes, fl[which])
         eng.close()
-    eng = packed(1, 1024)
-    us, nbytes = eng.time_kernel(5, 48)
-    kernels["packed: decode batch 1"]["attention, 1024 keys"] = frac(us, nbytes, 4 * 1024 * like["hidden"], fp32=True)
-    us, nbytes = eng.time_kernel(21, 48)
-    kernels["packed: prompt chunk of 512"]["attention, 512 queries, 1024 keys"] = frac(us, nbytes, 4 * 512 * 768 * like["hidden"])
-    eng.close()
+    if not like_name:
+        eng = packed(1, 1024)
+        us, nbytes = eng.time_kernel(5, 48)
+        kernels["packed: decode batch 1"]["attention, 1024 keys"] = frac(us, nbytes, 4 * 1024 * like["hidden"], fp32=True)
+        us, nbytes = eng.time_kernel(21, 48)
+        kernels["packed: prompt chunk of 512"]["attention, 512 queries, 1024 keys"] = frac(us, nbytes, 4 * 512 * 768 * like["hidden"])
+        eng.close()
     clocks = sampler.finish()
     line = {"metric": f"decode tokens/s of {args.block_model}, batch 1", "value": result["block model"]["decode"]["batch 1"]["tokens_per_s"], "unit": "tokens/s",
             "n_gpus": 1, "steps": steps, "warmup": warmup, "ms_per_step": result["block model"]["decode"]["batch 1"]["ms_per_step"], "higher_is_better": True,
-            "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "config": dict(shape, model=args.block_model, packed_like=like,
+            "vs_baseline": None, "dtype": "bf16", "data": "synthetic", "config": dict(shape, model=args.block_model, beside=like_name or like,
             l2="weights read per step exceed the 126 MB L2", timing="CUDA events around the device loop / the launches; prompts by the host clock around a synchronous call"),
             "throughput": result, "kernels": kernels, "peaks": {"hbm_GBps": peak, "bf16_TFLOPs": peak_tf, "source": peak_src}, "clocks": clocks}
     os.write(json_fd, (json.dumps(line) + "\n").encode())
@@ -374,7 +400,7 @@ def main():
     ap.add_argument("--planes", type=int, default=3, choices=[2, 3])
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-check", action="store_true", help="skip the in-run parity check against the golden fixtures")
-    ap.add_argument("--block-model", default=None, choices=["nezolix-w2048", "nezolix-w4096"], help="measure a block model instead of a workload")
+    ap.add_argument("--block-model", default=None, choices=["nezolix-w2048", "nezolix-w4096", "pizilix-w2048", "pizilix-w4096"], help="measure a block model instead of a workload")
     args = ap.parse_args()
     if args.block_model:
         return run_block(args)

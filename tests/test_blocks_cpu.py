@@ -36,6 +36,20 @@ def test_rotation_scaling_leaves_fast_pairs_and_divides_slow_ones():
     assert np.allclose(f[:5], g[:5]) and np.allclose(f[-1], g[-1] / 4) and np.isclose(amp, 1 + 0.1 * np.log(4.0))
 
 
+def test_chunked_mask_and_sink_of_the_plain_model():
+    assert [pb.seen_keys(p, {"size": 3}) for p in range(7)] == [0, 0, 0, 3, 3, 3, 6]
+    w = pb.sink_weights(np.array([[0.0, 0.0, 0.0], [50.0, 0.0, 0.0], [-50.0, -50.0, -50.0]]))
+    assert np.allclose(w[0], 0.25) and np.allclose(w[1], [1, 0, 0]) and w[2].sum() < 1e-20
+
+
+def test_recurrence_of_the_plain_model_keeps_its_variance():
+    """a^2 + (sqrt(1 - a^2))^2 = 1: white noise through an open input gate keeps unit variance."""
+    rng = np.random.default_rng(0)
+    u = rng.standard_normal((4000, 50))
+    out, _ = pb.gated_recurrence(u, np.full_like(u, 0.5), np.ones_like(u), rng.normal(-3, 1, 50), np.zeros(50))
+    assert 0.8 < out[500:].var() < 1.2
+
+
 def refused(pkg, tmp_path, match, change=None, tensors=None, name="odd"):
     cfg, t = bm.make(bm.CONFIGS[name])
     cfg = copy.deepcopy(cfg)
@@ -74,6 +88,18 @@ def test_model_folder_errors(pkg, tmp_path):
     refused(pkg, tmp_path, "l2.mix.uv has an unexpected shape", setter("layers", 2, "mixer", "vdim", value=10))
     refused(pkg, tmp_path, "l0.mix.dq.norm is missing", tensors=lambda t: t.pop("l0.mix.dq.norm"))
     refused(pkg, tmp_path, "w1 is missing", tensors=lambda t: t.pop("l1.mix.w1"))
+    def piz(match, change=None, tensors=None):
+        refused(pkg, tmp_path, match, change, tensors, name="piz_odd")
+
+    piz("unknown mixer 'wkv'", setter("layers", 1, "type", value="wkv"))
+    piz("heads must be a multiple of kv_heads", setter("layers", 0, "mixer", "kv_heads", value=4))
+    piz("vdim must equal dim", setter("layers", 0, "mixer", "vdim", value=10))
+    piz("rot.dims exceeds dim", setter("layers", 0, "mixer", "rot", "dims", value=22))
+    piz("rot.dims must be even", setter("layers", 0, "mixer", "rot", "dims", value=5))
+    piz("width must be a multiple of blocks", setter("layers", 1, "mixer", "blocks", value=5))
+    piz("missing field 'scale'", lambda c: c["layers"][0]["mixer"].pop("scale"))
+    piz("l1.mix.conv has an unexpected shape", setter("layers", 1, "mixer", "conv", value=4))
+    piz("l3.mix.ri.b is missing", tensors=lambda t: t.pop("l3.mix.ri.b"))
     with pytest.raises(pkg.B200Error, match="cannot open"):
         pkg.Engine.from_model(str(tmp_path / "nowhere"))
     (tmp_path / "m" / "config.json").write_text('{"architecture": "Nezolix", "layers": [}')

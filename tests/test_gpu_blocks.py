@@ -95,17 +95,93 @@ MECHANISMS = {  # one layer, one mechanism; the rest of the model is as plain as
     "wkv": [bm.wkv(ff=0)],
     "feed-forward": [bm.latent(window=1, ff=77)],
 }
+PIZILIX_MECHANISMS = {
+    "attention": [bm.attention(ff=0)],
+    "attention, rotation of the whole head": [bm.attention(ff=0, dim=16, rot={"base": 9.0, "dims": 16})],
+    "attention, one head each": [bm.attention(ff=0, heads=4, kv_heads=4, chunk=33)],
+    "attention, vectorised": [bm.attention(ff=0, heads=4, kv_heads=2, dim=32, chunk=40, rot={"base": 50.0, "dims": 16})],
+    "attention, yarn": [bm.attention(ff=0, dim=24, chunk=50, rot=bm.CHUNK_YARN)],
+    "attention, everything seen": [bm.attention(ff=0, chunk=0)],
+    "recurrence": [bm.rglru(ff=0)],
+    "recurrence, wide blocks": [bm.rglru(ff=0, width=192, blocks=1, conv=4)],
+    "feed-forward, silu": [bm.attention(chunk=1, ff=77)],
+}
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("name", list(MECHANISMS))
+@pytest.mark.parametrize("name", [*MECHANISMS, *PIZILIX_MECHANISMS])
 def test_each_mechanism_alone(pkg, case, name, dtype):
-    c = case(name.replace(" ", "_").replace(",", ""), cfg=bm.config(MECHANISMS[name]))
+    cfg = bm.config(MECHANISMS[name]) if name in MECHANISMS else bm.pizilix(PIZILIX_MECHANISMS[name])
+    c = case(name.replace(" ", "_").replace(",", ""), cfg=cfg)
     toks = bm.tokens(c.cfg, 70)
     ref = c.plain(toks)
     sess = pkg.Sessions(engine(pkg, c, dtype))
     assert err(feed(sess, 0, toks, [70]), ref) < c.limit(dtype, toks)
     assert err(feed(sess, 1, toks, [33] + [1] * 37), ref) < c.limit(dtype, toks)
+
+
+MISTAKES = {  # planted in the plain model: what a missing or wrong piece would do to the logits
+    "no sink": ("sink_weights", lambda s: np.exp(s - s.max(-1, keepdims=True)) / np.exp(s - s.max(-1, keepdims=True)).sum(-1, keepdims=True)),
+    "no cap on scores": ("softcap", None),
+    "sliding instead of chunked": ("seen_keys", lambda p, mask: max(0, p - mask["size"] + 1) if mask else 0),
+    "no rotation": ("rotate", lambda x, positions, rot: x),
+    "conv without history": ("causal_conv", lambda x, w, b, before: (x * w[:, -1] + b, before)),
+    "first token unscaled": ("gated_recurrence", None),
+    "relu for silu": ("silu", lambda z: np.maximum(z, 0)),
+}
+
+
+@pytest.mark.parametrize("name", list(MISTAKES))
+def test_mistakes_would_show(pkg, case, name, monkeypatch):
+    """The engine agrees with the plain model, and a plain model with one mistake does not."""
+    c = case("piz_mistakes", cfg=bm.pizilix([bm.attention(scale=1.0), bm.rglru(), bm.attention(chunk=20, scale=1.0)], loop={"start": 0, "stop": 2, "times": 2}))
+    toks = bm.tokens(c.cfg, 60)
+    ref, limit = c.plain(toks), c.limit("bfloat16", toks)
+    got = pkg.Sessions(engine(pkg, c, "bfloat16")).feed(0, toks, range(60))
+    assert err(got, ref) < limit
+    what, wrong = MISTAKES[name]
+    if name == "no cap on scores":
+        right = pb.softcap
+        wrong = lambda z, cap: z if cap == 6.0 else right(z, cap)
+    if name == "first token unscaled":
+        right_rec = pb.gated_recurrence
+
+        def wrong(u, r, i, lam, S):  # starts where the first token's state comes out as i u
+            a = np.exp(-8 * r[0] * np.logaddexp(0, lam))
+            return right_rec(u, r, i, lam, (1 - np.sqrt(1 - a * a)) / a * i[0] * u[0])
+    monkeypatch.setattr(pb, what, wrong)
+    assert err(pb.PlainModel(c.cfg, c.tensors).run(toks), ref) > 2 * limit
+
+
+def test_embedding_joins_every_further_pass(pkg, case):
+    """With one pass, or with layers unrolled under other names, the embedding is not added again: both differ from the loop."""
+    c = case("piz_mistakes", cfg=bm.pizilix([bm.attention(scale=1.0), bm.rglru(), bm.attention(chunk=20, scale=1.0)], loop={"start": 0, "stop": 2, "times": 2}))
+    toks = bm.tokens(c.cfg, 40)
+    unrolled = copy.deepcopy(c.cfg)
+    unrolled["loop"] = None
+    unrolled["layers"] = [c.cfg["layers"][l] for l in pb.layer_runs(c.cfg)]
+    t = {k: v for k, v in c.tensors.items() if not k.startswith("l")}
+    for i, l in enumerate(pb.layer_runs(c.cfg)):
+        t.update({f"l{i}." + k.split(".", 1)[1]: v for k, v in c.tensors.items() if k.startswith(f"l{l}.")})
+    assert err(pb.PlainModel(unrolled, t).run(toks), c.plain(toks)) > 0.1
+    from pathlib import Path
+    u = Case(pb.write_model(Path(c.folder).parent / "unrolled", unrolled, t), unrolled, t)
+    for x in (c, u):
+        sess = pkg.Sessions(engine(pkg, x, "float32"))
+        assert err(feed(sess, 0, toks, [21] + [1] * 19), x.plain(toks)) < 1e-4
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_residual_stream_of_one_token_pizilix(pkg, case, dtype):
+    """The same for a loop that adds the embedding again: what is handed in counts as the embedding."""
+    c = case("piz_odd")
+    eng = engine(pkg, c, dtype)
+    trace = []
+    ref = pb.PlainModel(c.cfg, c.tensors).run([42], trace)
+    x = eng.lookup_embedding(42)
+    logits = eng.forward(x, 0)
+    assert np.abs(x - trace[-1][0]).max() < (1e-4 if dtype == "float32" else 5e-2) * np.abs(trace[-1]).max()
+    assert err(logits[None], ref) < c.limit(dtype, [42])
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
@@ -124,7 +200,7 @@ def test_residual_stream_of_one_token(pkg, case, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("sizes", [(2,), (3, 2), (7, 1, 16), (64, 65, 3), (31,)])
-@pytest.mark.parametrize("name", ["odd", "aligned"])
+@pytest.mark.parametrize("name", ["odd", "aligned", "piz_odd", "piz_aligned"])
 def test_portions_of_several_sizes(pkg, case, name, sizes, dtype):
     c = case(name)
     toks = bm.tokens(c.cfg, 170)
@@ -138,7 +214,7 @@ def test_small_chunks_and_wrapping_rings(pkg, case, dtype, chunk, monkeypatch):
     """A prompt longer than a chunk is cut by the engine; the windowed caches are rings of window - 1 + chunk rows, which
     wrap many times here, in prompts and in decoding."""
     monkeypatch.setenv("B200_PREFILL_CHUNK", str(chunk))
-    for name in ("odd", "aligned"):
+    for name in ("odd", "aligned", "piz_odd", "piz_aligned"):
         c = case(name)
         toks = bm.tokens(c.cfg, 230)
         sess = pkg.Sessions(engine(pkg, c, dtype))
@@ -168,6 +244,83 @@ def test_window_edges(pkg, case, window, dtype):
     sess = pkg.Sessions(engine(pkg, c, dtype))
     for sid, cuts in enumerate(([150], [90] + [1] * 60, bm.cuts_of(150, 2, 5, 64, 1))):
         assert err(feed(sess, sid, toks, cuts), ref) < limit
+        sess.end(sid)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("chunk", [1, 2, 16, 63, 64, 65])
+def test_chunk_edges(pkg, case, chunk, dtype):
+    """The same for chunked masks: chunks one smaller or larger must be told apart, and so must chunks counted from where a
+    portion starts (positions restarting there)."""
+    cfg = bm.pizilix([bm.attention(chunk=chunk, ff=0), bm.attention(chunk=chunk, heads=4, kv_heads=1, dim=32, rot={"base": 40.0, "dims": 16}, ff=0)])
+    c = case(f"chunk{chunk}", sharp=3.0, cfg=cfg)
+    toks = bm.tokens(c.cfg, 150)
+    ref = c.plain(toks)
+    limit = c.limit(dtype, toks)
+    for off in (-1, 1):
+        if chunk + off < 1:
+            continue
+        wrong = copy.deepcopy(c.cfg)
+        for l in wrong["layers"]:
+            l["mixer"]["mask"]["size"] = chunk + off
+        assert err(pb.PlainModel(wrong, c.tensors).run(toks), ref) > 3 * limit
+    sess = pkg.Sessions(engine(pkg, c, dtype))
+    for sid, cuts in enumerate(([150], [90] + [1] * 60, bm.cuts_of(150, 2, 5, 64, 1))):
+        assert err(feed(sess, sid, toks, cuts), ref) < limit
+        sess.end(sid)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+@pytest.mark.parametrize("heads", [(2, 1, 32), (40, 2, 12)])
+def test_a_far_key_in_its_chunk(pkg, case, heads, dtype):
+    """An early token's key stands out for late queries until their chunk ends: in prompts, in decoding, and (many splits of the
+    context) at the splits' edges. The sink's share of the weight shows in the queries that see nothing alike."""
+    n, chunk, early = 660, 300, 305
+    H, G, D = heads
+    c = case(f"far_chunk{H}", cfg=bm.pizilix([bm.attention(heads=H, kv_heads=G, dim=D, chunk=chunk, scale=0.02, cap=30.0, rot={"base": 10.0, "dims": 4}, ff=0)]))
+    t = {k: v.copy() for k, v in c.tensors.items()}
+    W = c.cfg["width"]
+    t["embed"][:, :2] = 0
+    t["embed"][1], t["embed"][2] = np.eye(W)[0], np.eye(W)[1]
+    t["l0.norm1"][:] = 0
+    t["l0.mix.k"][:, 0] = 0
+    t["l0.mix.k"][5::D, 0] = 4
+    t["l0.mix.q"][:, 1] = 0
+    t["l0.mix.q"][5::D, 1] = 8
+    t = {k: pb.bf16_round(v) for k, v in t.items()}
+    from pathlib import Path
+    c2 = Case(pb.write_model(Path(c.folder).parent / f"far_chunk{H}b", c.cfg, t), c.cfg, t)
+    toks = [3 + v % (c.cfg["vocab"] - 3) for v in bm.tokens(c.cfg, n)]
+    toks[early] = 1
+    places = (early + 1, early + 64, early + 150, 2 * chunk - 1, 2 * chunk)
+    for p in places:
+        toks[p] = 2
+    ref = c2.plain(toks)
+    assert err(ref[places[-2]][None], ref[places[-1]][None]) > 0.3
+    sess = pkg.Sessions(engine(pkg, c2, dtype, max_ctx=700))
+    for sid, cuts in enumerate(([n], [early + 140] + [1] * (n - early - 140), bm.cuts_of(n, 50, 3))):
+        got = feed(sess, sid, toks, cuts)
+        for p in places:
+            assert err(got[p:p + 1], ref[p:p + 1]) < c2.limit(dtype, toks), p
+        sess.end(sid)
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_a_recurrence_that_remembers(pkg, case, dtype):
+    """Channels that hardly decay: what an early token left is still there hundreds of tokens later, across tiles and portions."""
+    c = case("remember", cfg=bm.pizilix([bm.rglru(width=72, blocks=2, conv=4, ff=0)]))
+    t = {k: v.copy() for k, v in c.tensors.items()}
+    t["l0.mix.lam"][:] = -9.0
+    t = {k: pb.bf16_round(v) for k, v in t.items()}
+    from pathlib import Path
+    c2 = Case(pb.write_model(Path(c.folder).parent / "remember2", c.cfg, t), c.cfg, t)
+    toks = bm.tokens(c.cfg, 330)
+    other = list(toks)
+    other[3] = (toks[3] + 1) % c.cfg["vocab"]
+    assert err(c2.plain(other)[-50:], c2.plain(toks)[-50:]) > 3e-3
+    sess = pkg.Sessions(engine(pkg, c2, dtype))
+    for sid, cuts in enumerate(([330], [65] * 5 + [5], [3, 127] + [1] * 200)):
+        assert err(feed(sess, sid, toks, cuts), c2.plain(toks)) < c2.limit(dtype, toks)
         sess.end(sid)
 
 
@@ -208,8 +361,9 @@ def test_a_far_key_among_hundreds(pkg, case, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_first_tokens_and_short_sequences(pkg, case, dtype):
-    c = case("odd")
+@pytest.mark.parametrize("name", ["odd", "piz_odd"])
+def test_first_tokens_and_short_sequences(pkg, case, name, dtype):
+    c = case(name)
     sess = pkg.Sessions(engine(pkg, c, dtype))
     for n in (1, 2, 3, 4, 5, 9):
         toks = bm.tokens(c.cfg, n, seed=50 + n)
@@ -219,8 +373,9 @@ def test_first_tokens_and_short_sequences(pkg, case, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_slots_that_are_freed_and_used_again(pkg, case, dtype):
-    c = case("odd")
+@pytest.mark.parametrize("name", ["odd", "piz_odd"])
+def test_slots_that_are_freed_and_used_again(pkg, case, name, dtype):
+    c = case(name)
     eng = engine(pkg, c, dtype, max_seqs=1)
     sess = pkg.Sessions(eng)
     long, short = bm.tokens(c.cfg, 140, seed=8), bm.tokens(c.cfg, 45, seed=9)
@@ -243,10 +398,11 @@ def test_slots_that_are_freed_and_used_again(pkg, case, dtype):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("batch", [2, 4, 7, 12, 19])
-def test_batches_of_unequal_requests_match_each_alone(pkg, case, dtype, batch):
+@pytest.mark.parametrize("name", ["odd", "piz_odd", "piz_aligned"])
+def test_batches_of_unequal_requests_match_each_alone(pkg, case, name, dtype, batch):
     """Prompts of unequal length in one call (runs share chunks), then joint decode steps in mixed slot order, on the
     matvec path (small batches) and on the row path (large ones)."""
-    c = case("odd")
+    c = case(name)
     eng = engine(pkg, c, dtype, max_seqs=batch + 2)
     lens = [3 + 11 * i % 37 for i in range(batch)]
     seqs = [bm.tokens(c.cfg, n + 6, seed=100 + i) for i, n in enumerate(lens)]
@@ -268,7 +424,7 @@ def test_batches_of_unequal_requests_match_each_alone(pkg, case, dtype, batch):
         assert err(tail[i:i + 1], refs[i][-1:]) < limit
 
 
-@pytest.mark.parametrize("name", ["odd", "wkv_only"])
+@pytest.mark.parametrize("name", ["odd", "wkv_only", "piz_odd", "piz_wide"])
 def test_greedy_generation(pkg, case, name):
     """The device-resident loop of a 32-bit engine chooses the plain model's ids."""
     c = case(name)
@@ -280,8 +436,9 @@ def test_greedy_generation(pkg, case, name):
     assert sess.live["g"][1] == 23 + 39
 
 
-def test_greedy_batch_and_penalty(pkg, case):
-    c = case("aligned")
+@pytest.mark.parametrize("name", ["aligned", "piz_aligned"])
+def test_greedy_batch_and_penalty(pkg, case, name):
+    c = case(name)
     eng = engine(pkg, c, "float32", max_seqs=3)
     prompts = [bm.tokens(c.cfg, n, seed=n) for n in (9, 30, 17)]
     first = eng.prefill_batch(prompts).argmax(axis=1)
@@ -306,18 +463,20 @@ def test_greedy_batch_and_penalty(pkg, case):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_long_decoding(pkg, case, dtype):
+@pytest.mark.parametrize("name", ["odd", "piz_odd"])
+def test_long_decoding(pkg, case, name, dtype):
     """400 decoded tokens: dozens of windows, and a recurrence that has forgotten its start."""
-    c = case("odd")
+    c = case(name)
     toks = bm.tokens(c.cfg, 420, seed=4)
     sess = pkg.Sessions(engine(pkg, c, dtype))
     assert err(feed(sess, 0, toks, [20] + [1] * 400), c.plain(toks)) < c.limit(dtype, toks)
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_results_do_not_depend_on_cuts_or_company(pkg, case, dtype):
+@pytest.mark.parametrize("name", ["yarn", "piz_aligned"])
+def test_results_do_not_depend_on_cuts_or_company(pkg, case, name, dtype):
     """The same tokens as one prompt, in portions, and beside other requests: equal beyond rounding."""
-    c = case("yarn")
+    c = case(name)
     toks = bm.tokens(c.cfg, 130, seed=12)
     eng = engine(pkg, c, dtype, max_seqs=4)
     a = eng.prefill(toks, slot=0)
@@ -329,8 +488,9 @@ def test_results_do_not_depend_on_cuts_or_company(pkg, case, dtype):
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
-def test_trace_replay_program(pkg, case, tmp_path, dtype):
-    c = case("odd")
+@pytest.mark.parametrize("name", ["odd", "piz_odd"])
+def test_trace_replay_program(pkg, case, tmp_path, name, dtype):
+    c = case(name)
     a, b = bm.tokens(c.cfg, 40, seed=1), bm.tokens(c.cfg, 12, seed=2)
     steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:25], "want": [0, 24]}], "end": []},
              {"step": 1, "entries": [{"id": "a", "tokens": a[25:39], "want": []}], "end": []},

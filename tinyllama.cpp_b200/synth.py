@@ -81,17 +81,31 @@ def quantize(ggml_type, x):
     return out
 
 
-# Block models of a real model's layer sizes: three latent-attention layers, then one WKV layer, repeated.
+# Block models of a real model's layer sizes. Nezolix: three latent-attention layers, then one WKV layer, repeated; Pizilix:
+# attention and RG-LRU layers in turn.
 BLOCK_SHAPES = {
-    "nezolix-w2048": dict(width=2048, ff=5632, vocab=32000, n_layers=8, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=256,
+    "pizilix-w2048": dict(design="Pizilix", width=2048, ff=5632, vocab=32000, n_layers=8, heads=16, kv_heads=4, dim=128, rot_dims=64, window=1024,
+                          lru_width=2048, lru_blocks=16, conv=4),
+    "pizilix-w4096": dict(design="Pizilix", width=4096, ff=11008, vocab=32000, n_layers=8, heads=32, kv_heads=8, dim=128, rot_dims=64, window=1024,
+                          lru_width=4096, lru_blocks=16, conv=4),
+    "nezolix-w2048": dict(design="Nezolix", width=2048, ff=5632, vocab=32000, n_layers=8, heads=16, dim=128, rot_dim=64, vdim=128, q_rank=768, kv_rank=256,
                           window=1024, wkv_heads=32, wkv_dim=64, decay_rank=64),
-    "nezolix-w4096": dict(width=4096, ff=11008, vocab=32000, n_layers=8, heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512,
+    "nezolix-w4096": dict(design="Nezolix", width=4096, ff=11008, vocab=32000, n_layers=8, heads=32, dim=128, rot_dim=64, vdim=128, q_rank=1536, kv_rank=512,
                           window=1024, wkv_heads=64, wkv_dim=64, decay_rank=64),
 }
 
 
 def block_config(shape):
     s = BLOCK_SHAPES[shape] if isinstance(shape, str) else shape
+    if s["design"] == "Pizilix":
+        mlp = {"kind": "dense", "ff": s["ff"]}
+        attn = {"type": "attention", "mlp": mlp,
+                "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5, "softcap": 50.0,
+                          "mask": {"size": s["window"]},
+                          "rot": {"base": 10000.0, "dims": s["rot_dims"], "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+        lru = {"type": "rglru", "mlp": mlp, "mixer": {"width": s["lru_width"], "blocks": s["lru_blocks"], "conv": s["conv"]}}
+        return {"architecture": "Pizilix", "width": s["width"], "vocab": s["vocab"], "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "loop": None,
+                "layers": [lru if l % 2 else attn for l in range(s["n_layers"])]}
     attn = {"type": "latent_attention", "mlp": {"kind": "dense", "ff": s["ff"]},
             "mixer": {"heads": s["heads"], "dim": s["dim"], "rot_dim": s["rot_dim"], "vdim": s["vdim"], "q_rank": s["q_rank"], "kv_rank": s["kv_rank"],
                       "scale": (s["dim"] + s["rot_dim"]) ** -0.5, "mask": {"size": s["window"]},
@@ -101,36 +115,45 @@ def block_config(shape):
             "layers": [wkv if l % 4 == 3 else attn for l in range(s["n_layers"])]}
 
 
-def block_tensors(cfg, decay_rank):
+def block_tensors(cfg, decay_rank=0):
     """(name, shape) of every tensor of a block model."""
     W = cfg["width"]
+    pizilix = cfg["architecture"] == "Pizilix"
     out = [("embed", (cfg["vocab"], W))]
     for i, l in enumerate(cfg["layers"]):
         L, m = f"l{i}.", l["mixer"]
-        H, D = m["heads"], m["dim"]
-        out += [(L + "norm1", (W,)), (L + "norm1b", (W,))]
+        H, D = m.get("heads"), m.get("dim")
+        out += [(L + "norm1", (W,))] + ([] if pizilix else [(L + "norm1b", (W,))])
         if l["type"] == "latent_attention":
             out += [(L + "mix." + n, s) for n, s in (
                 ("dq", (m["q_rank"], W)), ("dq.norm", (m["q_rank"],)), ("uq", (H * (D + m["rot_dim"]), m["q_rank"])), ("dkv", (m["kv_rank"] + m["rot_dim"], W)),
                 ("dkv.norm", (m["kv_rank"],)), ("uk", (H * D, m["kv_rank"])), ("uv", (H * m["vdim"], m["kv_rank"])), ("g", (H * m["vdim"], W)), ("o", (W, H * m["vdim"])))]
+        elif l["type"] == "attention":
+            out += [(L + "mix.q", (H * D, W)), (L + "mix.k", (m["kv_heads"] * D, W)), (L + "mix.o", (W, H * D))]
+        elif l["type"] == "rglru":
+            N, B = m["width"], m["blocks"]
+            S = N // B
+            out += [(L + "mix." + n, s) for n, s in (
+                ("y", (N, W)), ("y.b", (N,)), ("x", (N, W)), ("x.b", (N,)), ("conv", (N, m["conv"])), ("conv.b", (N,)), ("ra", (B, S, S)), ("ra.b", (B, S)),
+                ("ri", (B, S, S)), ("ri.b", (B, S)), ("lam", (N,)), ("o", (W, N)))]
         else:
             out += [(L + "mix.mu." + n, (W,)) for n in "rkvgw"] + [(L + "mix." + n, (H * D, W)) for n in "rkvg"]
             out += [(L + "mix." + n, s) for n, s in (("w1", (decay_rank, W)), ("w2", (H * D, decay_rank)), ("w0", (H * D,)), ("u", (H, D)), ("norm", (H * D,)), ("o", (W, H * D)))]
         if l["mlp"]:
             ff = l["mlp"]["ff"]
-            out += [(L + "norm2", (W,)), (L + "norm2b", (W,)), (L + "mlp.gate", (ff, W)), (L + "mlp.up", (ff, W)), (L + "mlp.down", (W, ff))]
-    return out + [("final.norm", (W,)), ("head", (cfg["vocab"], W))]
+            out += [(L + "norm2", (W,))] + ([] if pizilix else [(L + "norm2b", (W,))]) + [(L + "mlp.gate", (ff, W)), (L + "mlp.up", (ff, W)), (L + "mlp.down", (W, ff))]
+    return out + [("final.norm", (W,))] + ([] if pizilix else [("head", (cfg["vocab"], W))])
 
 
 def write_block_model(folder, shape, seed=1234, sigma=0.02):
     """Writes config.json and model.safetensors of a BLOCK_SHAPES entry: N(0, sigma) matrices (slices of one seeded block of
-    16 Mi values at seeded offsets), unit norms, token-shift mixes in [0, 1), decay biases around -3."""
+    16 Mi values at seeded offsets), unit norms, token-shift mixes in [0, 1), decay biases around -3 (WKV) and -5 (RG-LRU)."""
     os.makedirs(folder, exist_ok=True)
     s = BLOCK_SHAPES[shape] if isinstance(shape, str) else shape
     cfg = block_config(shape)
     with open(os.path.join(folder, "config.json"), "w") as f:
         json.dump(cfg, f)
-    names = block_tensors(cfg, s["decay_rank"])
+    names = block_tensors(cfg, s.get("decay_rank", 0))
     head, at = {}, 0
     for name, shp in names:
         n = int(np.prod(shp)) * 2
@@ -149,9 +172,11 @@ def write_block_model(folder, shape, seed=1234, sigma=0.02):
         for name, shp in names:
             n = int(np.prod(shp))
             if "norm" in name:
-                f.write(bits(np.ones(n)).tobytes())
+                f.write(bits(np.zeros(n) if s["design"] == "Pizilix" else np.ones(n)).tobytes())
             elif ".mu." in name:
                 f.write(bits(rng.uniform(0, 1, n)).tobytes())
+            elif name.endswith(".lam"):
+                f.write(bits(rng.normal(-5, 1, n)).tobytes())
             elif name.endswith(".w0"):
                 f.write(bits(rng.normal(-3, 1, n)).tobytes())
             else:
