@@ -40,8 +40,6 @@ __device__ __forceinline__ float rotated(const float* v, int i, const float* rop
   return (i & 1) ? v[i] * c + v[i - 1] * s : v[i] * c - v[i + 1] * s;
 }
 
-// tanh from one exponential: 1 - 2 / (1 + e^(2x)), absolute error of a few 2^-24 whatever x is
-__device__ __forceinline__ float tanh_by_exp(float x) { return 1.0f - __fdividef(2.0f, 1.0f + exp2f(x * 2.8853900817779268f)); }
 // cap * tanh(s / cap), or s itself without a cap
 __device__ __forceinline__ float capped_score(float s, float cap) { return cap > 0.f ? cap * tanhf(s / cap) : s; }
 
@@ -95,10 +93,11 @@ struct SplitStats {
 // brings a key's row into shared memory, one warp per row (columns beyond the row must come out as zeros; cp.async allowed);
 // scores run over columns ks0 .., the weighted sum over the first 8 * tiles columns: o[i] = this warp's column tile
 // 2 (warp + 8 (i / 2)) + i % 2 for heads g and g + 8. score(s) turns a product into a score. Ends with a block barrier, the
-// statistics complete in st (sums per warp; every warp holds the same maxima).
-template <int TW, typename LoadRow, typename Score>
-__device__ __forceinline__ void split_attend(const SplitTiles& m, SplitStats& st, int k_begin, int k_end, int ks0, int tiles, LoadRow load_row, Score score,
-                                             float (&o)[TW][4]) {
+// statistics complete in st (sums per warp; every warp holds the same maxima). queries() fills Qh and Ql; it runs while the
+// first rows are on their way.
+template <int TW, typename Queries, typename LoadRow, typename Score>
+__device__ __forceinline__ void split_attend(const SplitTiles& m, SplitStats& st, int k_begin, int k_end, int ks0, int tiles, Queries queries, LoadRow load_row,
+                                             Score score, float (&o)[TW][4]) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
   const int RS = m.RS, PS = LAS_KEYS + 8;
 #pragma unroll
@@ -106,13 +105,14 @@ __device__ __forceinline__ void split_attend(const SplitTiles& m, SplitStats& st
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;  // heads g and g + 8
   for (int kt = k_begin; kt < k_end; kt += LAS_KEYS) {
     const int nk = min(LAS_KEYS, k_end - kt);
-    __syncthreads();
+    if (kt > k_begin) __syncthreads();
     for (int r = warp; r < LAS_KEYS; r += LAS_WARPS) {
       __nv_bfloat16* d = m.Ks + r * RS;
       if (r < nk) load_row(kt + r, d);
       else
         for (int c = lane; c < m.EP >> 3; c += 32) *reinterpret_cast<uint4*>(d + 8 * c) = make_uint4(0, 0, 0, 0);
     }
+    if (kt == k_begin) queries();
     pfa_cp_wait_all();
     __syncthreads();
     // scores of this warp's 8 keys
@@ -238,6 +238,7 @@ struct PromptAttnParams {
   int gate_stride;
   const RunDesc* runs;
   int heads, dim, rot_dim, rot0, vdim;
+  int wave;                  // blocks that start together, one per SM
   KeyMask mask;
   float scale, softcap;      // softcap: see capped_score
   int sink;                  // one more term exp(0) in the softmax denominator
@@ -251,12 +252,19 @@ __host__ __device__ __forceinline__ size_t lap_smem_bytes(int dim, int rot, int 
   return ((size_t)(LAP_Q + LAP_K) * lap_qk_stride(dim, rot) + (size_t)LAP_K * (vp + 8)) * 2;
 }
 
-// grid = (query blocks of the longest run, heads, runs). VP = value columns per head rounded up to 32, 64, 128 or 256.
+// grid = (query blocks of the longest run * heads, 1, runs). VP = value columns per head rounded up to 32, 64, 128 or 256.
 template <int VP>
 __global__ void __launch_bounds__(LAP_THREADS, VP <= 128 ? 2 : 1) prompt_attn_kernel(const PromptAttnParams p) {
   extern __shared__ __align__(16) unsigned char lap_smem[];
   const RunDesc run = p.runs[blockIdx.z];
-  const int q0 = blockIdx.x * LAP_Q, h = blockIdx.y;
+  // later queries may see more keys: the heaviest blocks come first, and every second wave of blocks runs through the order
+  // backwards, so that blocks that share an SM add up to about the same
+  int order = blockIdx.x;
+  {
+    const int wave = order / p.wave, first = wave * p.wave;
+    if (wave & 1) order = first + min(p.wave, (int)gridDim.x - first) - 1 - (order - first);
+  }
+  const int q0 = (gridDim.x / p.heads - 1 - order / p.heads) * LAP_Q, h = order % p.heads;
   if (q0 >= run.len) return;
   const int E = p.dim + p.rot_dim, EP = (E + 15) / 16 * 16, QS = EP + 8;
   constexpr int VS = VP + 8, NT_O = VP / 8;
@@ -310,59 +318,66 @@ __global__ void __launch_bounds__(LAP_THREADS, VP <= 128 ? 2 : 1) prompt_attn_ke
   }
   const int qpos0 = run.start + q0;                       // position of the block's first query
   const int kfirst = p.mask.first(qpos0), klast = qpos0 + nq - 1;
-  const int base = run.start - run.hist;                  // position of the run's first context row
   const int my0 = qpos0 + warp * 16 + g, my1 = my0 + 8;   // this thread's two query positions
-  const int low0 = p.mask.first(my0), low1 = p.mask.first(my1);  // and the first keys they see
   float o[NT_O][4];
 #pragma unroll
   for (int i = 0; i < NT_O; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   // a sink is a key of score 0 without a value: it is there from the start (sums are shared by the four lanes of a row)
   float m0 = p.sink ? 0.f : -INFINITY, m1 = m0, l0 = p.sink && t == 0 ? 1.f : 0.f, l1 = l0;
   constexpr float LOG2E = 1.4426950408889634f;
-  const float sc2 = p.scale * LOG2E;
-  auto row_of = [&](int key) { return p.ring ? (size_t)(key % p.ring) : (size_t)(run.ctx0 + key - base); };
+  const float sc2 = p.scale * LOG2E, cap2 = p.softcap * LOG2E, to_tanh = p.softcap > 0.f ? 2.f * LOG2E * p.scale / p.softcap : 0.f;
+  const int wfirst = qpos0 + warp * 16, whigh = min(wfirst + 15, klast), wlow = p.mask.first(wfirst), wlast = p.mask.first(wfirst + 15);  // of the warp's queries
+  const int base = run.start - run.hist;                  // contiguous context: position of its first row
+  auto first_row = [&](int kt) { return p.ring ? kt % p.ring : run.ctx0 + kt - base; };
+  auto row_of = [&](int row0, int r) { return p.ring && row0 + r >= p.ring ? row0 + r - p.ring : row0 + r; };  // r rows further
+  // 16-byte pieces of a tile: a thread keeps its column and takes every k_rows-th (v_rows-th) row
+  constexpr int CV = VP >> 3, V_ROWS = LAP_THREADS / CV;
+  const int ce = EP >> 3, k_rows = LAP_THREADS / ce, kr0 = tid / ce, kc = tid - kr0 * ce;
+  const bool k_rot = kc >= p.rot0 >> 3 && kc < rot1 >> 3, k_has = kc < E >> 3;
+  const __nv_bfloat16* k_src = k_rot ? rotated_keys + 8 * kc - p.rot0 : keys + 8 * kc;
+  const int k_ld = k_rot ? p.kr_stride : p.kv_stride;
 
   // Key and value tiles have one buffer each: the next key tile is requested as soon as this one's scores are done, the
   // next value tile after this one's products, so each copy runs under the other half of the work.
   auto load_k = [&](int kt) {
-    const int nk = min(LAP_K, klast - kt + 1);
+    const int nk = min(LAP_K, klast - kt + 1), row0 = first_row(kt);
     if (vec) {
-      const int ce = EP >> 3, c0 = p.rot0 >> 3, c1 = rot1 >> 3, cn = E >> 3;
-      for (int r = warp; r < LAP_K; r += LAP_WARPS) {
-        const size_t row = r < nk ? row_of(kt + r) : 0;
-        const __nv_bfloat16* kv = keys + row * p.kv_stride;
-        const __nv_bfloat16* kr = rotated_keys + row * p.kr_stride;
-        for (int c = lane; c < ce; c += 32) {
-          __nv_bfloat16* d = Ks + r * QS + 8 * c;
-          if (r < nk && c < cn) pfa_cp16(d, c >= c0 && c < c1 ? kr + 8 * (c - c0) : kv + 8 * c);
+      if (kr0 < k_rows)
+        for (int r = kr0; r < LAP_K; r += k_rows) {
+          __nv_bfloat16* d = Ks + r * QS + 8 * kc;
+          if (r < nk && k_has) pfa_cp16(d, k_src + (size_t)row_of(row0, r) * k_ld);
           else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
         }
-      }
     } else {
       for (int i = tid; i < LAP_K * EP; i += LAP_THREADS) {
         const int r = i / EP, c = i - r * EP;
         __nv_bfloat16 v = __float2bfloat16(0.f);
-        if (r < nk && c < E) v = c >= p.rot0 && c < rot1 ? rotated_keys[row_of(kt + r) * p.kr_stride + c - p.rot0] : keys[row_of(kt + r) * p.kv_stride + c];
+        if (r < nk && c < E) {
+          const size_t row = row_of(row0, r);
+          v = c >= p.rot0 && c < rot1 ? rotated_keys[row * p.kr_stride + c - p.rot0] : keys[row * p.kv_stride + c];
+        }
         Ks[r * QS + c] = v;
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
   auto load_v = [&](int kt) {
-    const int nk = min(LAP_K, klast - kt + 1);
+    const int nk = min(LAP_K, klast - kt + 1), row0 = first_row(kt);
     if (vec) {
-      constexpr int CV = VP >> 3;
-      const int cvn = p.vdim >> 3;
-      for (int i = tid; i < LAP_K * CV; i += LAP_THREADS) {
-        const int r = i / CV, c = i % CV;
+      const int c = tid % CV;
+      const bool has = c < p.vdim >> 3;
+      const __nv_bfloat16* src = values + 8 * c;
+#pragma unroll
+      for (int i = 0; i < LAP_K / V_ROWS; ++i) {
+        const int r = tid / CV + i * V_ROWS;
         __nv_bfloat16* d = Vs + r * VS + 8 * c;
-        if (r < nk && c < cvn) pfa_cp16(d, values + row_of(kt + r) * p.kv_stride + 8 * c);
+        if (r < nk && has) pfa_cp16(d, src + (size_t)row_of(row0, r) * p.kv_stride);
         else *reinterpret_cast<uint4*>(d) = make_uint4(0, 0, 0, 0);
       }
     } else {
       for (int i = tid; i < LAP_K * VP; i += LAP_THREADS) {
         const int r = i / VP, c = i - r * VP;
-        Vs[r * VS + c] = r < nk && c < p.vdim ? values[row_of(kt + r) * p.kv_stride + c] : __float2bfloat16(0.f);
+        Vs[r * VS + c] = r < nk && c < p.vdim ? values[(size_t)row_of(row0, r) * p.kv_stride + c] : __float2bfloat16(0.f);
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
@@ -373,82 +388,95 @@ __global__ void __launch_bounds__(LAP_THREADS, VP <= 128 ? 2 : 1) prompt_attn_ke
     asm volatile("cp.async.wait_group 1;" ::: "memory");  // the key tile; its value tile may still be on its way
     __syncthreads();
     // scores: 16 queries x 64 keys per warp
+    const bool sees = kt <= whigh && kt + LAP_K > wlow;  // some query of this warp sees some key of the tile
     float s[8][4];
+    if (sees) {
 #pragma unroll
-    for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
-    for (int ks = 0; ks < EP; ks += 16) {
-      uint32_t a[4];
-      pfa_ldm4(a, Qs + (warp * 16 + (lane & 15)) * QS + ks + (lane >> 4) * 8);
+      for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.f;
+      for (int ks = 0; ks < EP; ks += 16) {
+        uint32_t a[4];
+        pfa_ldm4(a, Qs + (warp * 16 + (lane & 15)) * QS + ks + (lane >> 4) * 8);
 #pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {  // 16 keys: two 8-key fragments
-        uint32_t kb[4];
-        pfa_ldm4(kb, Ks + (nt * 16 + (lane & 7) + (lane >> 4) * 8) * QS + ks + ((lane >> 3) & 1) * 8);
-        lap_mma(s[2 * nt], a, kb[0], kb[1]);
-        lap_mma(s[2 * nt + 1], a, kb[2], kb[3]);
+        for (int nt = 0; nt < 4; ++nt) {  // 16 keys: two 8-key fragments
+          uint32_t kb[4];
+          pfa_ldm4(kb, Ks + (nt * 16 + (lane & 7) + (lane >> 4) * 8) * QS + ks + ((lane >> 3) & 1) * 8);
+          lap_mma(s[2 * nt], a, kb[0], kb[1]);
+          lap_mma(s[2 * nt + 1], a, kb[2], kb[3]);
+        }
       }
     }
     __syncthreads();  // every warp has read the key tile
     if (kt + LAP_K <= klast) load_k(kt + LAP_K);
     else asm volatile("cp.async.commit_group;" ::: "memory");  // keeps one group per step
-    if (p.softcap > 0.f) {
-      const float to_tanh = p.scale / p.softcap, from_tanh = p.softcap * LOG2E;
+    if (sees) {
+      if (p.softcap > 0.f) {  // cap * tanh(x / cap) with tanh(z) = 1 - 2 / (1 + e^(2z)), then to base 2
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
+        for (int i = 0; i < 8; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[i][e] = from_tanh * tanh_by_exp(s[i][e] * to_tanh);
-    } else {
+          for (int e = 0; e < 4; ++e) s[i][e] = fmaf(-2.f * cap2, rcp_fast(1.f + ex2_fast(s[i][e] * to_tanh)), cap2);
+      } else {
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
+        for (int i = 0; i < 8; ++i)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) s[i][e] *= sc2;
-    }
-    float n0 = m0, n1 = m1;
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-#pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        const int key = kt + 8 * i + 2 * t + e;
-        s[i][e] = key <= my0 && key >= low0 ? s[i][e] : -INFINITY;
-        s[i][2 + e] = key <= my1 && key >= low1 ? s[i][2 + e] : -INFINITY;
-        n0 = fmaxf(n0, s[i][e]);
-        n1 = fmaxf(n1, s[i][2 + e]);
+          for (int e = 0; e < 4; ++e) s[i][e] *= sc2;
       }
-    }
+      if (kt + LAP_K - 1 > wfirst || kt < wlast) {  // not every query of the warp sees every key
+        const int low0 = p.mask.first(my0), low1 = p.mask.first(my1);
 #pragma unroll
-    for (int x = 1; x < 4; x <<= 1) {
-      n0 = fmaxf(n0, __shfl_xor_sync(0xffffffffu, n0, x));
-      n1 = fmaxf(n1, __shfl_xor_sync(0xffffffffu, n1, x));
-    }
-    // a row that has seen no key yet keeps -infinity: subtract 0 then, every weight is exp2(-inf) = 0
-    const float z0 = n0 == -INFINITY ? 0.f : n0, z1 = n1 == -INFINITY ? 0.f : n1;
-    const float f0 = exp2f(m0 - z0), f1 = exp2f(m1 - z1);
-    m0 = n0; m1 = n1;
-    l0 *= f0; l1 *= f1;
+        for (int i = 0; i < 8; ++i)
 #pragma unroll
-    for (int i = 0; i < NT_O; ++i) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
+          for (int e = 0; e < 2; ++e) {
+            const int key = kt + 8 * i + 2 * t + e;
+            if (key > my0 || key < low0) s[i][e] = -INFINITY;
+            if (key > my1 || key < low1) s[i][2 + e] = -INFINITY;
+          }
+      }
+      float n0 = m0, n1 = m1;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+      for (int i = 0; i < 8; ++i) {
+        n0 = fmaxf(n0, fmaxf(s[i][0], s[i][1]));
+        n1 = fmaxf(n1, fmaxf(s[i][2], s[i][3]));
+      }
 #pragma unroll
-      for (int e = 0; e < 2; ++e) {
-        s[i][e] = exp2f(s[i][e] - z0);
-        s[i][2 + e] = exp2f(s[i][2 + e] - z1);
-        l0 += s[i][e];
-        l1 += s[i][2 + e];
+      for (int x = 1; x < 4; x <<= 1) {
+        n0 = fmaxf(n0, __shfl_xor_sync(0xffffffffu, n0, x));
+        n1 = fmaxf(n1, __shfl_xor_sync(0xffffffffu, n1, x));
+      }
+      // a row that has seen no key yet keeps -infinity: subtract 0 then, every weight is 2^-inf = 0
+      const float z0 = n0 == -INFINITY ? 0.f : n0, z1 = n1 == -INFINITY ? 0.f : n1;
+      if (__any_sync(0xffffffffu, n0 != m0 || n1 != m1)) {
+        const float f0 = ex2_fast(m0 - z0), f1 = ex2_fast(m1 - z1);
+        l0 *= f0; l1 *= f1;
+#pragma unroll
+        for (int i = 0; i < NT_O; ++i) { o[i][0] *= f0; o[i][1] *= f0; o[i][2] *= f1; o[i][3] *= f1; }
+      }
+      m0 = n0; m1 = n1;
+#pragma unroll
+      for (int i = 0; i < 8; ++i) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          s[i][e] = ex2_fast(s[i][e] - z0);
+          s[i][2 + e] = ex2_fast(s[i][2 + e] - z1);
+          l0 += s[i][e];
+          l1 += s[i][2 + e];
+        }
       }
     }
     asm volatile("cp.async.wait_group 1;" ::: "memory");  // the value tile
     __syncthreads();
     // weighted values
+    if (sees) {
 #pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-      const uint32_t a[4] = {pack_bf2(s[2 * kk][0], s[2 * kk][1]), pack_bf2(s[2 * kk][2], s[2 * kk][3]), pack_bf2(s[2 * kk + 1][0], s[2 * kk + 1][1]),
-                             pack_bf2(s[2 * kk + 1][2], s[2 * kk + 1][3])};
+      for (int kk = 0; kk < 4; ++kk) {
+        const uint32_t a[4] = {pack_bf2(s[2 * kk][0], s[2 * kk][1]), pack_bf2(s[2 * kk][2], s[2 * kk][3]), pack_bf2(s[2 * kk + 1][0], s[2 * kk + 1][1]),
+                               pack_bf2(s[2 * kk + 1][2], s[2 * kk + 1][3])};
 #pragma unroll
-      for (int nt = 0; nt < NT_O / 2; ++nt) {
-        uint32_t vb[4];
-        pfa_ldm4t(vb, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + nt * 16 + (lane >> 4) * 8);
-        lap_mma(o[2 * nt], a, vb[0], vb[1]);
-        lap_mma(o[2 * nt + 1], a, vb[2], vb[3]);
+        for (int nt = 0; nt < NT_O / 2; ++nt) {
+          uint32_t vb[4];
+          pfa_ldm4t(vb, Vs + (kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * VS + nt * 16 + (lane >> 4) * 8);
+          lap_mma(o[2 * nt], a, vb[0], vb[1]);
+          lap_mma(o[2 * nt + 1], a, vb[2], vb[3]);
+        }
       }
     }
     __syncthreads();  // every warp has read the value tile

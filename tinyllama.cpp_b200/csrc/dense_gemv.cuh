@@ -24,13 +24,26 @@ enum : int { ACT_NONE = 0, ACT_SIGMOID, ACT_SILU, ACT_TANH, ACT_DECAY, ACT_GELU,
 
 __host__ __device__ __forceinline__ bool act_is_glu(int act) { return act >= ACT_RELU_GLU; }
 __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf(-z)); }
-__device__ __forceinline__ float gelu_tanh_f(float z) { return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z))); }
+// 2^x and 1 / x of the special-function unit: FP32 to within two units in the last place, tiny results become zero
+__device__ __forceinline__ float ex2_fast(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rcp_fast(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// z * sigmoid(w): SiLU with w = z; GELU (tanh form, 0.5 z (1 + tanh(v)) = z sigmoid(2v)) with w = 2v
+__device__ __forceinline__ float swish_f(float z, float w) { return z * rcp_fast(1.0f + ex2_fast(-1.4426950408889634f * w)); }
+__device__ __forceinline__ float gelu_tanh_f(float z) { return swish_f(z, 1.5957691216057308f * (z + 0.044715f * z * z * z)); }
 __device__ __forceinline__ float softcap_f(float z, float cap) { return cap * tanhf(z / cap); }
 // v: the row's product with its bias added; arg: the cap of ACT_SOFTCAP
 __device__ __forceinline__ float dense_act(int act, float v, float arg) {
   switch (act) {
     case ACT_SIGMOID: return sigmoid_f(v);
-    case ACT_SILU: return v * sigmoid_f(v);
+    case ACT_SILU: return swish_f(v, v);
     case ACT_TANH: return tanhf(v);
     case ACT_DECAY: return expf(-expf(v));
     case ACT_GELU: return gelu_tanh_f(v);
@@ -38,7 +51,7 @@ __device__ __forceinline__ float dense_act(int act, float v, float arg) {
     default: return v;
   }
 }
-__device__ __forceinline__ float glu_act(int act, float gate, float up) { return (act == ACT_SILU_GLU ? gate * sigmoid_f(gate) : fmaxf(gate, 0.f)) * up; }
+__device__ __forceinline__ float glu_act(int act, float gate, float up) { return (act == ACT_SILU_GLU ? swish_f(gate, gate) : fmaxf(gate, 0.f)) * up; }
 
 __host__ __device__ __forceinline__ int pad8(int n) { return (n + 7) & ~7; }
 // Gate and up rows of a gated feed-forward share one matrix: eight gate rows, then the same eight up rows.

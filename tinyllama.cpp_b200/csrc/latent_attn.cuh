@@ -453,18 +453,20 @@ __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentS
   const int k_begin = lo + split * chunk, k_end = min(pos + 1, k_begin + chunk);
   const __nv_bfloat16* cache = p.cache + (size_t)p.slots[b] * p.cap * p.crow;
   const int nh = min(LAS_HEADS, p.heads - h0), ce = m.EP >> 3, cc = p.crow >> 3;
-  for (int r = warp; r < LAS_HEADS; r += LAS_WARPS) {
-    const size_t at = ((size_t)b * p.heads + h0 + min(r, nh - 1)) * p.qrow;
-    for (int c = lane; c < ce; c += 32) {
-      if (r < nh) {
-        pfa_cp16(m.Qh + r * m.RS + 8 * c, p.q_hi + at + 8 * c);
-        pfa_cp16(m.Ql + r * m.RS + 8 * c, p.q_lo + at + 8 * c);
-      } else {
-        *reinterpret_cast<uint4*>(m.Qh + r * m.RS + 8 * c) = make_uint4(0, 0, 0, 0);
-        *reinterpret_cast<uint4*>(m.Ql + r * m.RS + 8 * c) = make_uint4(0, 0, 0, 0);
+  auto queries = [&] {
+    for (int r = warp; r < LAS_HEADS; r += LAS_WARPS) {
+      const size_t at = ((size_t)b * p.heads + h0 + min(r, nh - 1)) * p.qrow;
+      for (int c = lane; c < ce; c += 32) {
+        if (r < nh) {
+          pfa_cp16(m.Qh + r * m.RS + 8 * c, p.q_hi + at + 8 * c);
+          pfa_cp16(m.Ql + r * m.RS + 8 * c, p.q_lo + at + 8 * c);
+        } else {
+          *reinterpret_cast<uint4*>(m.Qh + r * m.RS + 8 * c) = make_uint4(0, 0, 0, 0);
+          *reinterpret_cast<uint4*>(m.Ql + r * m.RS + 8 * c) = make_uint4(0, 0, 0, 0);
+        }
       }
     }
-  }
+  };
   const int tiles = p.kvp >> 3;  // 8-column tiles of the weighted sum; a warp takes pairs of them
   float o[TW][4];
   auto load_row = [&](int key, __nv_bfloat16* d) {
@@ -474,7 +476,7 @@ __global__ void __launch_bounds__(LAS_THREADS) latent_split_kernel(const LatentS
       else *reinterpret_cast<uint4*>(d + 8 * c) = make_uint4(0, 0, 0, 0);
     }
   };
-  split_attend<TW>(m, st, k_begin, k_end, 0, tiles, load_row, [](float s) { return s; }, o);
+  split_attend<TW>(m, st, k_begin, k_end, 0, tiles, queries, load_row, [](float s) { return s; }, o);
   const size_t row = ((size_t)b * p.heads + h0) * p.nsplit + split;
   if (tid < nh) {
     float* ml = p.part_ml + (row + (size_t)tid * p.nsplit) * 2;

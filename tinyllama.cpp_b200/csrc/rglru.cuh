@@ -43,11 +43,20 @@ struct RgLruParams {
   int out_stride;
 };
 
-// a and sqrt(1 - a^2) from the gate's product r (before the sigmoid)
+__device__ __forceinline__ float gate_sigmoid(float z) { return rcp_fast(1.0f + ex2_fast(-1.4426950408889634f * z)); }
+// a and sqrt(1 - a^2) from the gate's product r (before the sigmoid). 1 - a^2 = 1 - e^x with x = 2 log a loses digits for
+// small x: there it is -x times the series of (e^x - 1) / x.
 __device__ __forceinline__ void rglru_decay(float r, float decay, float& a, float& norm) {
-  const float log_a = -decay * sigmoid_f(r);
-  a = expf(log_a);
-  norm = sqrtf(-expm1f(2.0f * log_a));
+  const float log_a = -decay * gate_sigmoid(r), x = 2.0f * log_a;
+  a = ex2_fast(1.4426950408889634f * log_a);
+  float series = fmaf(x, 1.f / 5040.f, 1.f / 720.f);
+  series = fmaf(x, series, 1.f / 120.f);
+  series = fmaf(x, series, 1.f / 24.f);
+  series = fmaf(x, series, 1.f / 6.f);
+  series = fmaf(x, series, 0.5f);
+  series = fmaf(x, series, 1.f);
+  const float left = x > -0.5f ? -x * series : fmaf(-a, a, 1.f);
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(norm) : "f"(left));
 }
 
 constexpr int RGS_THREADS = 256, RGS_WARPS = 8;
@@ -133,7 +142,7 @@ __global__ void __launch_bounds__(RGS_THREADS) rglru_step_kernel(const RgLruPara
   float a, norm;
   rglru_decay(r + p.ra_b[ch], p.decay[ch], a, norm);
   float* S = p.state + (size_t)p.slots[b0 + n] * p.wp + ch;
-  const float in = norm * sigmoid_f(g + p.ri_b[ch]) * rgs_u[n * up + c];
+  const float in = norm * gate_sigmoid(g + p.ri_b[ch]) * rgs_u[n * up + c];
   const float s = fmaf(a, p.positions[b0 + n] > 0 ? *S : 0.f, in);
   *S = s;
   static_cast<O*>(p.out)[(size_t)(b0 + n) * p.out_stride + ch] = to_operand<O>(s * p.y[(size_t)(b0 + n) * p.stride + ch]);
@@ -176,18 +185,23 @@ __global__ void __launch_bounds__(RGP_THREADS) rglru_gates_kernel(const RgLruPar
   };
   // this thread's share of the convolution: one channel, RGP_SEG consecutive tokens
   const int cc = tid % RGP_TILE, ct = tid / RGP_TILE * RGP_SEG;
-  auto input = [&](int ch, int t) {  // x of token t of the run (t < 0: before it)
-    if (t >= 0) return p.x[(size_t)(run.row0 + t) * p.stride + ch];
+  auto before = [&](int ch, int t) {  // x of token t < 0 of the run
     const int pos = run.start + t;
     return pos >= 0 ? ring[(size_t)(pos % p.taps) * p.wp + ch] : 0.f;
   };
-  float win[RGP_SEG + RGP_TAPS - 1];  // win[j]: token t0 + ct + j - (RGP_TAPS - 1)
+  const float* xs = p.x + (size_t)(run.row0 + t0 + ct) * p.stride;
+  const int left = run.len - t0 - ct;  // tokens of the run from this thread's first one on
+  float win[RGP_SEG + RGP_TAPS - 1];   // win[j]: token j - (RGP_TAPS - 1) from there
   auto fetch_x = [&](int step) {
-    const int c = step * RGP_TILE + cc;
+    const int c = step * RGP_TILE + cc, ch = base + c;
+    const bool ok = c < p.bs;
 #pragma unroll
-    for (int j = 0; j < RGP_SEG + RGP_TAPS - 1; ++j) {
-      const int back = RGP_TAPS - 1 - j, t = t0 + ct - back;  // tokens further back than the taps reach are not kept
-      win[j] = c < p.bs && t < run.len && back < p.taps ? input(base + c, t) : 0.f;
+    for (int j = 0; j < RGP_SEG; ++j) win[RGP_TAPS - 1 + j] = ok && j < left ? xs[(size_t)j * p.stride + ch] : 0.f;
+#pragma unroll
+    for (int back = 1; back < RGP_TAPS; ++back) {  // tokens further back than the taps reach are not kept
+      float v = 0.f;
+      if (ok && left > 0 && back < p.taps) v = t0 + ct >= back ? xs[ch - (ptrdiff_t)back * p.stride] : before(ch, t0 + ct - back);
+      win[RGP_TAPS - 1 - back] = v;
     }
   };
   auto store_u = [&](int step) {
@@ -197,21 +211,33 @@ __global__ void __launch_bounds__(RGP_THREADS) rglru_gates_kernel(const RgLruPar
     float* f = reinterpret_cast<float*>(stage);
     const bool ok = c < p.bs;
     const float bias = ok ? p.conv_b[ch] : 0.f;
+    auto put = [&](int j, float u) {
+      if (F32) f[(ct + j) * RGP_LD + cc] = u;
+      else split_bf16(u, hi[(ct + j) * RGP_LD + cc], lo[(ct + j) * RGP_LD + cc]);
+      if (step == piece) Us[(ct + j) * RGP_FLD + cc] = u;
+    };
+    if (p.taps > RGP_TAPS) {  // any number of taps, straight from memory
+#pragma unroll 1
+      for (int j = 0; j < RGP_SEG; ++j) {
+        float u = bias;
+        if (ok && j < left)
+          for (int k = 0; k < p.taps; ++k) {
+            const float x = t0 + ct + j >= k ? xs[ch + (ptrdiff_t)(j - k) * p.stride] : before(ch, t0 + ct + j - k);
+            u = fmaf(p.conv[(size_t)(p.taps - 1 - k) * p.wp + ch], x, u);
+          }
+        put(j, u);
+      }
+      return;
+    }
     float w[RGP_TAPS];
 #pragma unroll
     for (int k = 0; k < RGP_TAPS; ++k) w[k] = ok && k < p.taps ? p.conv[(size_t)(p.taps - 1 - k) * p.wp + ch] : 0.f;  // k tokens back
 #pragma unroll
-    for (int j = 0; j < RGP_SEG; ++j) {
+    for (int j = 0; j < RGP_SEG; ++j) {  // values of tokens beyond the run stay unused
       float u = bias;
 #pragma unroll
       for (int k = 0; k < RGP_TAPS; ++k) u = fmaf(w[k], win[j + RGP_TAPS - 1 - k], u);
-      const int t = t0 + ct + j;
-      if (ok && t < run.len)
-        for (int k = RGP_TAPS; k < p.taps; ++k) u = fmaf(p.conv[(size_t)(p.taps - 1 - k) * p.wp + ch], input(ch, t - k), u);
-      if (t >= run.len) u = 0.f;
-      if (F32) f[(ct + j) * RGP_LD + cc] = u;
-      else split_bf16(u, hi[(ct + j) * RGP_LD + cc], lo[(ct + j) * RGP_LD + cc]);
-      if (step == piece) Us[(ct + j) * RGP_FLD + cc] = u;
+      put(j, u);
     }
   };
 
@@ -278,48 +304,46 @@ __global__ void __launch_bounds__(RGP_THREADS) rglru_gates_kernel(const RgLruPar
   }
   __syncthreads();  // the operand tiles are free, u is complete
 
-  // ---- decays and inputs of the recurrence, in place of the operand tiles and of u ----
-  float* As = reinterpret_cast<float*>(rgp_smem);
+  // ---- recurrence inside the tile: 16 tokens of a channel per thread, then the segments before this one ----
+  float *Rs = reinterpret_cast<float*>(rgp_smem), *Is = Rs + RGP_TILE * RGP_FLD;  // gate products [token][channel]
 #pragma unroll
-  for (int e = 0; e < 2; ++e) {
-    const int c = r0 + g + 8 * e, ch = base + c0 + c;
-    if (c0 + c >= p.bs) continue;
-    const float rb = p.ra_b[ch], ib = p.ri_b[ch], dec = p.decay[ch];
+  for (int i = 0; i < 4; ++i)
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
-#pragma unroll
-      for (int j = 0; j < 2; ++j) {
-        const int at = (n0 + 8 * i + 2 * t + j) * RGP_FLD + c;
-        float a, norm;
-        rglru_decay(acc[0][i][2 * e + j] + rb, dec, a, norm);
-        As[at] = a;
-        Us[at] *= norm * sigmoid_f(acc[1][i][2 * e + j] + ib);
-      }
-  }
+    for (int e = 0; e < 4; ++e) {
+      const int at = (n0 + 8 * i + 2 * t + (e & 1)) * RGP_FLD + r0 + g + 8 * (e >> 1);
+      Rs[at] = acc[0][i][e];
+      Is[at] = acc[1][i][e];
+    }
   __syncthreads();
-  // ---- recurrence inside the tile: 16 tokens per thread, then the segments before this one ----
+  const int last = min(ct + RGP_SEG, nt);
+  const bool mine = c0 + cc < p.bs;
+  const int ch = base + c0 + (mine ? cc : 0);
+  const float rb = p.ra_b[ch], ib = p.ri_b[ch], dec = p.decay[ch];
   float P = 1.f, Q = 0.f;
-  for (int j = ct; j < min(ct + RGP_SEG, nt); ++j) {
-    const float a = As[j * RGP_FLD + cc];
+#pragma unroll 2
+  for (int j = ct; j < last; ++j) {  // the pair of every token, in place of its gate product and u
+    const int at = j * RGP_FLD + cc;
+    float a, norm;
+    rglru_decay(Rs[at] + rb, dec, a, norm);
     P *= a;
-    Q = fmaf(a, Q, Us[j * RGP_FLD + cc]);
-    As[j * RGP_FLD + cc] = P;
-    Us[j * RGP_FLD + cc] = Q;
+    Q = fmaf(a, Q, norm * gate_sigmoid(Is[at] + ib) * Us[at]);
+    Rs[at] = P;
+    Us[at] = Q;
   }
   seg_p[tid] = P;
   seg_q[tid] = Q;
   __syncthreads();
-  if (c0 + cc >= p.bs) return;
-  const int ch = base + c0 + cc;
+  if (!mine) return;
   P = 1.f;
   Q = t0 == 0 && run.start > 0 ? p.state[(size_t)run.slot * p.wp + ch] : 0.f;  // the run's first tile starts from the slot's state
   for (int s = cc; s < tid; s += RGP_TILE) {
     Q = fmaf(seg_p[s], Q, seg_q[s]);
     P *= seg_p[s];
   }
-  for (int j = ct; j < min(ct + RGP_SEG, nt); ++j) {
+#pragma unroll 4
+  for (int j = ct; j < last; ++j) {
     const size_t row = (size_t)(run.row0 + t0 + j) * p.pq_stride + ch;
-    const float pj = As[j * RGP_FLD + cc];
+    const float pj = Rs[j * RGP_FLD + cc];
     p.P[row] = P * pj;
     p.Q[row] = fmaf(pj, Q, Us[j * RGP_FLD + cc]);
   }

@@ -87,7 +87,7 @@ __global__ void __launch_bounds__(LAS_THREADS) shared_kv_decode_kernel(const Sha
   const SplitTiles m(skv_smem, p.crow);
   pdl_launch_dependents();
   pdl_wait();
-  const int pos = p.positions[b];
+  const int pos = p.positions[b], slot = p.slots[b];
   if (pos < 0 || pos >= p.max_ctx) {  // nothing is read or appended for this sequence
     if (tid == 0 && p.error_flag) *reinterpret_cast<volatile int*>(p.error_flag) = 3;
     return;
@@ -96,14 +96,16 @@ __global__ void __launch_bounds__(LAS_THREADS) shared_kv_decode_kernel(const Sha
   const int chunk = ((nkeys + p.nsplit - 1) / p.nsplit + LAS_KEYS - 1) / LAS_KEYS * LAS_KEYS;
   const int k_begin = lo + split * chunk, k_end = min(pos + 1, k_begin + chunk);
   const int ce = m.EP >> 3, cc = p.crow >> 3;
-  __nv_bfloat16* cache = static_cast<__nv_bfloat16*>(p.cache) + ((size_t)p.slots[b] * p.kv_heads + g) * p.cap * p.crow;
+  __nv_bfloat16* cache = static_cast<__nv_bfloat16*>(p.cache) + ((size_t)slot * p.kv_heads + g) * p.cap * p.crow;
   const float* table = p.rope + (size_t)pos * p.pairs * 2;
-  if (k_begin < k_end)
-    for (int i = tid; i < LAS_HEADS * m.EP; i += LAS_THREADS) {
-      const int r = i / m.EP, c = i - r * m.EP;
-      const float v = r < nh && c < p.crow ? skv_query(p, p.q + (size_t)b * p.q_stride + (size_t)(h0 + r) * p.dim, table, c) * p.scale : 0.f;
-      split_bf16(v, m.Qh[r * m.RS + c], m.Ql[r * m.RS + c]);
+  auto queries = [&] {
+    for (int r = warp; r < LAS_HEADS; r += LAS_WARPS) {
+      const float* q = p.q + (size_t)b * p.q_stride + (size_t)(h0 + r) * p.dim;
+#pragma unroll 2
+      for (int c = lane; c < m.EP; c += 32)
+        split_bf16(r < nh && c < p.crow ? skv_query(p, q, table, c) * p.scale : 0.f, m.Qh[r * m.RS + c], m.Ql[r * m.RS + c]);
     }
+  };
   // the new token's row is made here, by every block whose run it lies in; one of them keeps it
   const float* key = p.k + (size_t)b * p.k_stride + g * p.dim;
   auto load_row = [&](int kp, __nv_bfloat16* d) {
@@ -124,7 +126,7 @@ __global__ void __launch_bounds__(LAS_THREADS) shared_kv_decode_kernel(const Sha
   const int tiles = p.vp >> 3;
   float o[TW][4];
   // whole 32-column steps in which every query is zero are left out
-  split_attend<TW>(m, st, k_begin, k_end, 2 * p.pairs / 32 * 32, tiles, load_row, [&](float s) { return capped_score(s, p.softcap); }, o);
+  split_attend<TW>(m, st, k_begin, k_end, 2 * p.pairs / 32 * 32, tiles, queries, load_row, [&](float s) { return capped_score(s, p.softcap); }, o);
 
   auto put = [&](int h, int c, float v) {
     if (c < p.dim) static_cast<O*>(p.out)[(size_t)b * p.out_stride + (size_t)(h0 + h) * p.dim + c] = to_operand<O>(v);
@@ -147,13 +149,15 @@ __global__ void __launch_bounds__(LAS_THREADS) shared_kv_decode_kernel(const Sha
     split_columns<TW>(o, tiles, nh, [&](int h, int c, float x, float y) {
       *reinterpret_cast<float2*>(p.part_o + (base + (size_t)h * p.nsplit + split) * p.vp + c) = make_float2(x, y);
     });
-  __threadfence();
   __syncthreads();
   int* ticket = p.tickets + (size_t)b * gridDim.y + blockIdx.y;
-  if (tid == 0) last_s = atomicAdd(ticket, 1) == p.nsplit - 1;
+  if (tid == 0) {  // the fence covers what the block's other threads wrote before the barrier
+    __threadfence();
+    last_s = atomicAdd(ticket, 1) == p.nsplit - 1;
+    __threadfence();
+  }
   __syncthreads();
   if (!last_s) return;
-  __threadfence();
   if (tid == 0) *ticket = 0;
   for (int h = warp; h < nh; h += LAS_WARPS) {  // weight of every run: exp(its max - the largest max) / total sum
     float mx[SKV_MAX_SPLITS / 32], l[SKV_MAX_SPLITS / 32], M = p.sink ? 0.f : -INFINITY, L = 0.f;
