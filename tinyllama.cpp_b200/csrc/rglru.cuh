@@ -59,6 +59,23 @@ __device__ __forceinline__ void rglru_decay(float r, float decay, float& a, floa
   asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(norm) : "f"(left));
 }
 
+// Sums N values over the warp (N a power of two up to 32): every lane gets the total of value lane % N.
+template <int N>
+__device__ __forceinline__ float lane_sums(float (&v)[N]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int s = N / 2; s > 0; s >>= 1)
+#pragma unroll
+    for (int j = 0; j < s; ++j) {
+      const bool up = lane & s;
+      const float send = up ? v[j] : v[j + s], keep = up ? v[j + s] : v[j];
+      v[j] = keep + __shfl_xor_sync(0xffffffffu, send, s);
+    }
+#pragma unroll
+  for (int s = N; s < 32; s <<= 1) v[0] += __shfl_xor_sync(0xffffffffu, v[0], s);
+  return v[0];
+}
+
 constexpr int RGS_THREADS = 256, RGS_WARPS = 8;
 constexpr int RGS_ROWS = 4;                        // channels per warp
 constexpr int RGS_CH = RGS_WARPS * RGS_ROWS;       // channels per block
@@ -88,27 +105,50 @@ __global__ void __launch_bounds__(RGS_THREADS) rglru_step_kernel(const RgLruPara
   };
   load(0);
   pdl_wait();
-  for (int i = tid; i < NB * up; i += RGS_THREADS) {
-    const int n = i / up, c = i - n * up, ch = base + c;
-    float u = 0.f;
-    if (n < nb && c < p.bs) {
-      const int pos = p.positions[b0 + n];
-      float* ring = p.ring + (size_t)p.slots[b0 + n] * p.taps * p.wp + ch;
-      const float x = p.x[(size_t)(b0 + n) * p.stride + ch];
-      u = fmaf(p.conv[(size_t)(p.taps - 1) * p.wp + ch], x, p.conv_b[ch]);
-      for (int k = 1; k < p.taps && k <= pos; ++k) u = fmaf(p.conv[(size_t)(p.taps - 1 - k) * p.wp + ch], ring[(size_t)((pos - k) % p.taps) * p.wp], u);
-      if (piece == 0) ring[(size_t)(pos % p.taps) * p.wp] = x;  // a row nobody reads in this launch
+  // what this lane finishes: channel (lane % 4) of sequence lane / 4
+  const int fn = lane / RGS_ROWS, fc = c0 + lane % RGS_ROWS, fch = base + fc;
+  const bool mine = fn < nb && fc < p.bs;
+  float old = 0.f, yv = 0.f, rb = 0.f, ib = 0.f, dec = 0.f;
+  float* S = nullptr;
+  if (mine) {
+    S = p.state + (size_t)p.slots[b0 + fn] * p.wp + fch;
+    if (p.positions[b0 + fn] > 0) old = *S;
+    yv = p.y[(size_t)(b0 + fn) * p.stride + fch];
+    rb = p.ra_b[fch]; ib = p.ri_b[fch]; dec = p.decay[fch];
+  }
+  int pos[NB];
+  float* ring[NB];
+#pragma unroll
+  for (int n = 0; n < NB; ++n) {
+    pos[n] = n < nb ? p.positions[b0 + n] : 0;
+    ring[n] = p.ring + (n < nb ? (size_t)p.slots[b0 + n] * p.taps * p.wp : 0) + base;
+  }
+  for (int c = tid; c < up; c += RGS_THREADS) {
+    const bool ok = c < p.bs;
+    const int ch = base + (ok ? c : 0);
+    const float w = p.conv[(size_t)(p.taps - 1) * p.wp + ch], bias = p.conv_b[ch];
+    float u[NB];
+#pragma unroll
+    for (int n = 0; n < NB; ++n) {
+      const float x = ok && n < nb ? p.x[(size_t)(b0 + n) * p.stride + ch] : 0.f;
+      u[n] = fmaf(w, x, bias);
+      if (piece == 0 && ok && n < nb) ring[n][(size_t)(pos[n] % p.taps) * p.wp + c] = x;  // a row nobody reads in this launch
     }
-    rgs_u[i] = u;
+    for (int k = 1; k < p.taps; ++k) {
+      const float wk = p.conv[(size_t)(p.taps - 1 - k) * p.wp + ch];
+#pragma unroll
+      for (int n = 0; n < NB; ++n)
+        if (ok && k <= pos[n]) u[n] = fmaf(wk, ring[n][(size_t)((pos[n] - k) % p.taps) * p.wp + c], u[n]);
+    }
+#pragma unroll
+    for (int n = 0; n < NB; ++n) rgs_u[n * up + c] = ok && n < nb ? u[n] : 0.f;
   }
   __syncthreads();
-  float acc[2][RGS_ROWS][NB];
+  float acc[2][RGS_ROWS * NB];  // [matrix][sequence * 4 + channel]
 #pragma unroll
   for (int m = 0; m < 2; ++m)
 #pragma unroll
-    for (int i = 0; i < RGS_ROWS; ++i)
-#pragma unroll
-      for (int n = 0; n < NB; ++n) acc[m][i][n] = 0.f;
+    for (int i = 0; i < RGS_ROWS * NB; ++i) acc[m][i] = 0.f;
   for (int it = 0; it * 32 < kc; ++it) {
     if (it) load(it);
     const int c = it * 32 + lane;
@@ -122,30 +162,20 @@ __global__ void __launch_bounds__(RGS_THREADS) rglru_step_kernel(const RgLruPara
 #pragma unroll
         for (int i = 0; i < RGS_ROWS; ++i) {
           const uint4 v = w[m][i];
-          float s = acc[m][i][n];
+          float s = acc[m][n * RGS_ROWS + i];
           s = fmaf(bf_lo(v.x), u[0], s); s = fmaf(bf_hi(v.x), u[1], s); s = fmaf(bf_lo(v.y), u[2], s); s = fmaf(bf_hi(v.y), u[3], s);
           s = fmaf(bf_lo(v.z), u[4], s); s = fmaf(bf_hi(v.z), u[5], s); s = fmaf(bf_lo(v.w), u[6], s); s = fmaf(bf_hi(v.w), u[7], s);
-          acc[m][i][n] = s;
+          acc[m][n * RGS_ROWS + i] = s;
         }
     }
   }
-  float r = 0.f, g = 0.f;  // lane = channel (lane & 3) of sequence lane >> 2
-#pragma unroll
-  for (int i = 0; i < RGS_ROWS; ++i)
-#pragma unroll
-    for (int n = 0; n < NB; ++n) {
-      const float s0 = warp_sum(acc[0][i][n]), s1 = warp_sum(acc[1][i][n]);
-      if (lane == n * RGS_ROWS + i) { r = s0; g = s1; }
-    }
-  const int n = lane / RGS_ROWS, c = c0 + lane % RGS_ROWS, ch = base + c;
-  if (n >= nb || c >= p.bs) return;
+  const float r = lane_sums(acc[0]), g = lane_sums(acc[1]);
+  if (!mine) return;
   float a, norm;
-  rglru_decay(r + p.ra_b[ch], p.decay[ch], a, norm);
-  float* S = p.state + (size_t)p.slots[b0 + n] * p.wp + ch;
-  const float in = norm * gate_sigmoid(g + p.ri_b[ch]) * rgs_u[n * up + c];
-  const float s = fmaf(a, p.positions[b0 + n] > 0 ? *S : 0.f, in);
+  rglru_decay(r + rb, dec, a, norm);
+  const float s = fmaf(a, old, norm * gate_sigmoid(g + ib) * rgs_u[fn * up + fc]);
   *S = s;
-  static_cast<O*>(p.out)[(size_t)(b0 + n) * p.out_stride + ch] = to_operand<O>(s * p.y[(size_t)(b0 + n) * p.stride + ch]);
+  static_cast<O*>(p.out)[(size_t)(b0 + fn) * p.out_stride + fch] = to_operand<O>(s * yv);
 }
 
 // ---- prompts -----------------------------------------------------------------------------------------------------
