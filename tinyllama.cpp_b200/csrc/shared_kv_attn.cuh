@@ -99,17 +99,24 @@ __global__ void __launch_bounds__(LAS_THREADS) shared_kv_decode_kernel(const Sha
   __nv_bfloat16* cache = static_cast<__nv_bfloat16*>(p.cache) + ((size_t)slot * p.kv_heads + g) * p.cap * p.crow;
   const float* table = p.rope + (size_t)pos * p.pairs * 2;
   auto queries = [&] {
-    for (int r = warp; r < LAS_HEADS; r += LAS_WARPS) {
-      const float* q = p.q + (size_t)b * p.q_stride + (size_t)(h0 + r) * p.dim;
-#pragma unroll 2
-      for (int c = lane; c < m.EP; c += 32)
-        split_bf16(r < nh && c < p.crow ? skv_query(p, q, table, c) * p.scale : 0.f, m.Qh[r * m.RS + c], m.Ql[r * m.RS + c]);
+    const int pieces = m.EP / 32;  // of 32 columns; those of the group's heads are shared out evenly over the warps
+    const float* q = p.q + (size_t)b * p.q_stride + (size_t)h0 * p.dim;
+#pragma unroll 4
+    for (int i = warp; i < nh * pieces; i += LAS_WARPS) {
+      const int r = i / pieces, c = (i - r * pieces) * 32 + lane;
+      split_bf16(c < p.crow ? skv_query(p, q + r * p.dim, table, c) * p.scale : 0.f, m.Qh[r * m.RS + c], m.Ql[r * m.RS + c]);
+    }
+    for (int i = nh * ce + tid; i < LAS_HEADS * ce; i += LAS_THREADS) {
+      const int r = i / ce, c = i - r * ce;
+      *reinterpret_cast<uint4*>(m.Qh + r * m.RS + 8 * c) = *reinterpret_cast<uint4*>(m.Ql + r * m.RS + 8 * c) = make_uint4(0, 0, 0, 0);
     }
   };
   // the new token's row is made here, by every block whose run it lies in; one of them keeps it
+  const int ring0 = k_begin % p.cap;
   const float* key = p.k + (size_t)b * p.k_stride + g * p.dim;
   auto load_row = [&](int kp, __nv_bfloat16* d) {
-    __nv_bfloat16* row = cache + (size_t)(kp % p.cap) * p.crow;
+    const int at = ring0 + kp - k_begin;  // fewer rows than the ring has: it wraps once at most
+    __nv_bfloat16* row = cache + (size_t)(at >= p.cap ? at - p.cap : at) * p.crow;
     if (kp == pos) {
       for (int c = lane; c < m.EP; c += 32) {
         const __nv_bfloat16 v = __float2bfloat16(c < p.crow ? skv_row(p, key, table, c) : 0.f);
@@ -125,8 +132,10 @@ __global__ void __launch_bounds__(LAS_THREADS) shared_kv_decode_kernel(const Sha
   };
   const int tiles = p.vp >> 3;
   float o[TW][4];
+  const float to_tanh = p.softcap > 0.f ? 2.8853900817779268f / p.softcap : 0.f;
+  auto score = [&](float s) { return p.softcap > 0.f ? fmaf(-2.f * p.softcap, rcp_fast(1.f + ex2_fast(s * to_tanh)), p.softcap) : s; };  // as in prompt_attn_kernel
   // whole 32-column steps in which every query is zero are left out
-  split_attend<TW>(m, st, k_begin, k_end, 2 * p.pairs / 32 * 32, tiles, queries, load_row, [&](float s) { return capped_score(s, p.softcap); }, o);
+  split_attend<TW>(m, st, k_begin, k_end, 2 * p.pairs / 32 * 32, tiles, queries, load_row, score, o);
 
   auto put = [&](int h, int c, float v) {
     if (c < p.dim) static_cast<O*>(p.out)[(size_t)b * p.out_stride + (size_t)(h0 + h) * p.dim + c] = to_operand<O>(v);
