@@ -22,9 +22,9 @@
 #include "gguf.h"
 #include "latent_attn.cuh"
 #include "misc.cuh"
-#include "tp.h"
 #include "rglru.cuh"
 #include "shared_kv_attn.cuh"
+#include "tp.h"
 #include "wkv.cuh"
 
 namespace b200 {
